@@ -156,7 +156,7 @@ int hb_sample(const float* logits, long long stride, const float* temperature, c
               void* stream);
 
 // A norm on a sublayer's output on its way into the residual stream: x += rmsnorm(y) * (offset + w); with w2 and h
-// also h = rmsnorm(x) * (offset2 + w2) for the next sublayer (post_norm.cu).  out = sa a + sb b over n floats.
+// also h = rmsnorm(x) * (offset2 + w2) for the next sublayer, with h alone h = x (post_norm.cu).  out = sa a + sb b over n floats.
 int hb_rmsnorm_add(const float* y, long long ldy, const float* w, float eps, float offset, float* x, long long ldx,
                    const float* w2, float eps2, float offset2, void* h, int h_dtype, long long ldh, int n_rows, int n, void* stream);
 int hb_scaled_sum(const float* a, float sa, const float* b, float sb, float* out, long long n, void* stream);
@@ -201,7 +201,7 @@ int hb_layernorm_add(const float* y, long long ldy, const float* y2, long long l
                      float eps, float* x, long long ldx, void* copy, int copy_dtype, long long ldc, int n_rows, int n, void* stream);
 int hb_convert(const float* x, void* out, int out_dtype, long long n, void* stream);
 // Attention over one cached latent per token (latent_attention.cu): the cache rows, and the per-head products around it
-int hb_latent_prepare(const float* proj, long long ldp, int n_heads, int d, int dr, int rank, int down_at, const float* c_weight, float eps,
+int hb_latent_prepare(const float* q, long long ldq_in, const float* down, long long ldd, int n_heads, int d, int dr, int rank, const float* c_weight, float eps,
                       const float* table, int rot, void* q_out, int q_dtype, long long ldq, int q_head, int q_rot_at, int q_copy, void* k_cache,
                       void* v_cache, int cache_dtype, const int* page_table, int pt_width, const int* tok_seq, const int* positions, int n_tokens,
                       int n_pages, int append, int* status, void* stream);
@@ -225,7 +225,7 @@ int hb_selective_scan(const void* u, int u_dtype, long long ldu, const float* bc
                       void* stream);
 // Mixture of experts (moe.cu)
 int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, int* experts, float* weights, int n_tokens, int width,
-                 int n_experts, int top, void* stream);
+                 int n_experts, int top, int scoring, void* stream);
 // tile_rows: hb_moe_tile_rows(tensor_cores), the rows of a plan tile of the products' variant (FP32 pipe, or mma.sync for
 // bfloat16 operands whose rows are multiples of 8 elements)
 int hb_moe_tile_rows(int tensor_cores);
@@ -233,7 +233,7 @@ int hb_moe_plan(const int* experts, int n_entries, int n_experts, int tile_rows,
 int hb_moe_max_tiles(int n_entries, int n_experts, int tile_rows);
 int hb_moe_glu(const void* h, int h_dtype, long long ldh, const void* w_gate, const void* w_up, int w_dtype, const int* offsets,
                const int* order, const int* tiles, int max_tiles, int top, void* act, int act_dtype, long long lda, int ff, int width,
-               float limit, float alpha, int tensor_cores, void* stream);
+               int unit, float limit, float alpha, const float* in_weights, int tensor_cores, void* stream);
 int hb_moe_down(const void* act, int act_dtype, long long lda, const void* w_down, int w_dtype, const int* offsets, const int* order,
                 const int* tiles, int max_tiles, int top, float* down, long long ldd, int width, int ff, int tensor_cores, void* stream);
 // experts non-null: entries whose expert number is n_real or more are identity experts (their result is the row of h)
@@ -260,13 +260,24 @@ int hb_scaled_add_norm(const float* y, long long ldy, float m, float* x, long lo
 int hb_normed_sum(const float* a, long long lda, const float* wa, const float* b, long long ldb, const float* wb, float eps, float* out,
                   long long ldo, int n_rows, int n, int accumulate, void* stream);
 // The recurrent memory per head with token-dependent decay (head_scan.cu): decay_mode 0 one scalar per (token, head) from a
-// step size, 1 one per (token, head, state index) from a sigmoid; chunk_len 0: one block walks a sequence's tokens, else
+// step size, 1 one per (token, head, state index) from a sigmoid, 2 a forget gate with a lower bound whose complement is the
+// input gate (kmat null); q_act 1: silu on q; chunk_len 0: one block walks a sequence's tokens, else
 // three launches with carry of n_seqs * max_chunks * heads * (2 * head_dim * n_state + (mode ? n_state : 1)) floats
 int hb_head_scan(const float* u, long long ldu, const float* kmat, long long ldk, const float* qmat, long long ldq, const float* z,
-                 long long ldz, const float* draw, long long ldd, const float* dbias, const float* a_log, float inv_tau,
-                 const float* dskip, float q_scale, float* state, long long state_stride, const int* state_slots, const int* seq_start,
+                 long long ldz, const float* draw, long long ldd, const float* dbias, const float* a_log, const float* lower,
+                 int q_act, float inv_tau, const float* dskip, float q_scale, float* state, long long state_stride, const int* state_slots, const int* seq_start,
                  void* out, int out_dtype, long long ldo, int n_seqs, int n_heads, int n_groups, int head_dim, int n_state,
                  int decay_mode, int chunk_len, int max_chunks, float* carry, long long carry_floats, void* stream);
+// Norms over equal parts of a row, alone and behind the sum of the stream and a gated sublayer's result (group_norm.cu):
+// x = norm(alpha x + sigmoid(gate + bias) * (the sum of n_sum rows of y per token)), copy = x in copy's dtype
+int hb_group_rmsnorm(const float* x, long long ldx, const float* w, float eps, int groups, void* out, int out_dtype, long long ldo,
+                     const int* rows, int n_rows, int n, void* stream);
+int hb_gated_sum_norm(float* x, long long ldx, float alpha, const float* y, long long ldy, int n_sum, const float* gate, long long ldg,
+                      const float* gate_bias, const float* w, float eps, int groups, void* copy, int copy_dtype, long long ldc, int n_rows, int n,
+                      void* stream);
+// out = gelu_tanh(s) * table[token][col0 ..], zeros in the columns dim .. n_out (token_side.cu)
+int hb_side_unit(const float* s, long long lds, const int* tokens, const void* table, int table_dtype, long long ldt, long long col0, int vocab,
+                 void* out, int out_dtype, long long ldo, int dim, int n_out, int n_tokens, int* status, void* stream);
 
 #ifdef __cplusplus
 }

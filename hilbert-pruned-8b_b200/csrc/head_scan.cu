@@ -1,5 +1,6 @@
 // A recurrent matrix memory per head whose decay depends on the token: the state-space form with one scalar
-// decay per (token, head), and the gated linear attention form with one decay per (token, head, key channel).
+// decay per (token, head), the gated linear attention form with one decay per (token, head, key channel), and the
+// forget-gate form, in which one minus that decay takes the place of the key.
 //
 // Per sequence, head h, value channel j (of P) and state index n (of N), all in 32-bit:
 //   S[j][n] <- a[t][h][n] S[j][n] + s[t][h] u[t][h][j] k[t][g(h)][n]          (evaluated as S + (a - 1) S + s u k)
@@ -7,6 +8,9 @@
 // with g(h) = h / (H / G) (G groups of heads share k and q).  The decay a and the input's factor s:
 //   mode 0 (scalar):  dt = softplus(dt_raw[t][h] + dt_bias[h]),  a = exp(-exp(A_log[h]) dt) for every n,  s = dt
 //   mode 1 (channel): a = sigmoid(a_raw[t][h][n] + a_bias[h][n]) ^ inv_tau = exp(-softplus(-(..)) inv_tau),  s = 1
+//   mode 2 (forget gate): a = l[h][n] + (1 - l[h][n]) sigmoid(a_raw[t][h][n] + a_bias[h][n]) with a lower bound l,  s = 1, and
+//                     k[t][h][n] = 1 - a = (1 - l) sigmoid(-(..)): made without a subtraction; kmat is not read
+// q may pass silu while it is staged (q_act).
 // a - 1 is made by expm1 from the decay's logarithm: with decays close to one, exp() rounded to 32 bits would be off by
 // percents of the distance to one, and that error would grow with every token.
 //
@@ -28,6 +32,7 @@
 #define HS_PAD 4            // floats between two lanes' runs of a staged row: the lanes' 16-byte loads then hit different banks
 
 __device__ __forceinline__ float hs_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float hs_silu(float z) { return z / (1.0f + expf(-z)); }
 
 // LANES threads own a value channel; each holds PER consecutive state indices (n = lane * PER + k) in registers, so that the
 // staged k, q and decay rows are read by 16-byte loads and the sum over n needs log2(LANES) shuffles per token.  Rows are
@@ -37,7 +42,7 @@ __global__ void __launch_bounds__(HS_THREADS, PER <= 8 ? 4 : 2)
 head_scan_kernel(const float* __restrict__ u, long long ldu, const float* __restrict__ kmat, long long ldk,
                  const float* __restrict__ qmat, long long ldq, const float* __restrict__ z, long long ldz,
                  const float* __restrict__ draw, long long ldd, const float* __restrict__ dbias, const float* __restrict__ a_log,
-                 float inv_tau, const float* __restrict__ dskip, float q_scale, float* __restrict__ state, long long state_stride,
+                 const float* __restrict__ lower, int q_act, float inv_tau, const float* __restrict__ dskip, float q_scale, float* __restrict__ state, long long state_stride,
                  const int* __restrict__ state_slots, const int* __restrict__ seq_start, TO* __restrict__ out, long long ldo,
                  int H, int G, int P, int N, int decay_mode, int pass, int chunk_len, int max_chunks, float* __restrict__ carry_L,
                  float* __restrict__ carry_log, const float* __restrict__ carry_S0) {
@@ -139,14 +144,14 @@ head_scan_kernel(const float* __restrict__ u, long long ldu, const float* __rest
         }
         // the tokens' k, q and decay inputs: HS_STAGE loads of a thread in flight before the first is used
         for (int i0 = tid; i0 < nt * NP; i0 += HS_THREADS * HS_STAGE) {
-            float kv[HS_STAGE], qv[HS_STAGE], dr[HS_STAGE];
+            float kv[HS_STAGE], qv[HS_STAGE], dr[HS_STAGE];      // (mode 2 keeps 1 - l where the keys would be)
 #pragma unroll
             for (int s8 = 0; s8 < HS_STAGE; s8++) {
                 const int i = i0 + s8 * HS_THREADS, r = i / NP, n = i - r * NP;
                 kv[s8] = qv[s8] = dr[s8] = 0.0f;
                 if (i < nt * NP && n < N) {
                     const size_t t = (size_t)(start + base + r);
-                    kv[s8] = kmat[t * ldk + (size_t)g * N + n];
+                    kv[s8] = decay_mode == 2 ? 1.0f - lower[(size_t)h * N + n] : kmat[t * ldk + (size_t)g * N + n];
                     qv[s8] = qmat[t * ldq + (size_t)g * N + n];
                     if (decay_mode) dr[s8] = draw[t * ldd + (size_t)h * N + n] + dbias[(size_t)h * N + n];
                 }
@@ -158,13 +163,17 @@ head_scan_kernel(const float* __restrict__ u, long long ldu, const float* __rest
                 const int at = r * RS + (n / PER) * (PER + HS_PAD) + n % PER;
                 if (decay_mode == 0) {
                     kv[s8] *= ds[r];
+                } else if (decay_mode == 2) {
+                    kv[s8] = n < N ? kv[s8] / (1.0f + expf(dr[s8])) : 0.0f;              // 1 - a
+                    if (sums_logs) ls[i] = log1pf(-kv[s8]);
+                    es[at] = -kv[s8];
                 } else {
                     const float lg = n < N ? -hs_softplus(-dr[s8]) * inv_tau : 0.0f;      // log(sigmoid) / tau
                     ls[i] = lg;
                     es[at] = expm1f(lg);
                 }
                 ks[at] = kv[s8];
-                qs[at] = qv[s8];
+                qs[at] = q_act ? hs_silu(qv[s8]) : qv[s8];
             }
         }
         for (int i = tid; i < nt * CH; i += HS_THREADS) {
@@ -282,7 +291,7 @@ static void hs_shape(int N, int P, long long grids, int& lanes, int& per) {
 
 extern "C" int hb_head_scan(const float* u, long long ldu, const float* kmat, long long ldk, const float* qmat, long long ldq,
                             const float* z, long long ldz, const float* draw, long long ldd, const float* dbias, const float* a_log,
-                            float inv_tau, const float* dskip, float q_scale, float* state, long long state_stride,
+                            const float* lower, int q_act, float inv_tau, const float* dskip, float q_scale, float* state, long long state_stride,
                             const int* state_slots, const int* seq_start, void* out, int out_dtype, long long ldo, int n_seqs,
                             int n_heads, int n_groups, int head_dim, int n_state, int decay_mode, int chunk_len, int max_chunks,
                             float* carry, long long carry_floats, void* stream) {
@@ -290,9 +299,11 @@ extern "C" int hb_head_scan(const float* u, long long ldu, const float* kmat, lo
     const int H = n_heads, G = n_groups, P = head_dim, N = n_state;
     HB_REQUIRE(n_seqs > 0 && H > 0 && G > 0 && P > 0 && N > 0 && H % G == 0 && H <= 65535, "head_scan: bad sizes");
     HB_REQUIRE(N <= 256, "head_scan: state size %d (up to 256 is built)", N);
-    HB_REQUIRE(decay_mode == 0 || decay_mode == 1, "head_scan: decay mode %d (0 scalar per head, 1 per state index)", decay_mode);
-    HB_REQUIRE(draw != nullptr && dbias != nullptr && (decay_mode == 1 || a_log != nullptr), "head_scan: the decay's inputs are missing");
-    HB_REQUIRE(ldu >= (long long)H * P && ldk >= (long long)G * N && ldq >= (long long)G * N && ldo >= (long long)H * P &&
+    HB_REQUIRE(decay_mode >= 0 && decay_mode <= 2, "head_scan: decay mode %d (0 scalar per head, 1 per state index, 2 forget gate)", decay_mode);
+    HB_REQUIRE(draw != nullptr && dbias != nullptr && (decay_mode != 0 || a_log != nullptr) && (decay_mode != 2 || lower != nullptr),
+               "head_scan: the decay's inputs are missing");
+    HB_REQUIRE(decay_mode == 2 ? G == H : kmat != nullptr, "head_scan: a forget gate has no keys and no groups, the other forms have keys");
+    HB_REQUIRE(ldu >= (long long)H * P && (decay_mode == 2 || ldk >= (long long)G * N) && ldq >= (long long)G * N && ldo >= (long long)H * P &&
                (z == nullptr || ldz >= (long long)H * P) && ldd >= (decay_mode ? (long long)H * N : (long long)H) &&
                state_stride >= (long long)H * P * N, "head_scan: rows are too short");
     HB_REQUIRE(out_dtype == HB_BF16 || out_dtype == HB_F32, "head_scan: unsupported output dtype %d", out_dtype);
@@ -322,7 +333,7 @@ extern "C" int hb_head_scan(const float* u, long long ldu, const float* kmat, lo
             }                                                                                                                           \
         }                                                                                                                               \
         hb_launch(head_scan_kernel<TO, L, PER>, dim3((P + ch - 1) / ch, H, n_seqs * (PASS == 0 ? 1 : max_chunks)), dim3(HS_THREADS), smem, s, \
-                  u, ldu, kmat, ldk, qmat, ldq, z, ldz, draw, ldd, dbias, a_log, inv_tau, dskip, q_scale, state, state_stride,           \
+                  u, ldu, kmat, ldk, qmat, ldq, z, ldz, draw, ldd, dbias, a_log, lower, q_act, inv_tau, dskip, q_scale, state, state_stride, \
                   state_slots, seq_start, (TO*)out, ldo, H, G, P, N, decay_mode, PASS, chunk_len, max_chunks, carry_L, carry_log,        \
                   (const float*)carry_S0);                                                                                              \
     }

@@ -20,7 +20,7 @@
 
 template <typename TQ>
 __global__ void __launch_bounds__(LP_THREADS)
-latent_prepare_kernel(const float* __restrict__ proj, long long ldp, int nh, int d, int dr, int rank, int down_at,
+latent_prepare_kernel(const float* __restrict__ q, long long ldq_in, const float* __restrict__ down, long long ldd, int nh, int d, int dr, int rank,
                       const float* __restrict__ c_weight, float eps, const float2* __restrict__ table, int rot,
                       TQ* __restrict__ q_out, long long ldq, int q_head, int q_rot_at, int q_copy, TQ* __restrict__ k_cache, TQ* __restrict__ v_cache,
                       const int* __restrict__ page_table, int pt_width, const int* __restrict__ tok_seq,
@@ -39,13 +39,13 @@ latent_prepare_kernel(const float* __restrict__ proj, long long ldp, int nh, int
         }
     }
     pdl_wait();
-    proj = pdl_fresh(proj);
+    q = pdl_fresh(q);
+    down = pdl_fresh(down);
     table = pdl_fresh(table);
-    const float* row = proj + (size_t)t * ldp;
     if (slot < nh) {
         // the rotated part of head `slot`'s query at column q_rot_at of the head's q_head columns: behind the rank numbers
         // that head_linear fills (q_copy 0), or behind the head's own unrotated part, copied here, with zeros up to q_head
-        const float* src = row + (size_t)slot * (d + dr) + d;
+        const float* src = q + (size_t)t * ldq_in + (size_t)slot * (d + dr) + d;
         TQ* head = q_out + (size_t)t * ldq + (size_t)slot * q_head;
         TQ* dst = head + q_rot_at;
         if (q_copy > 0) {
@@ -62,7 +62,7 @@ latent_prepare_kernel(const float* __restrict__ proj, long long ldp, int nh, int
         for (int i = rot + tid; i < dr; i += LP_THREADS) dst[i] = from_f32<TQ>(src[i]);
         return;
     }
-    const float* src = row + down_at;
+    const float* src = down + (size_t)t * ldd;
     float ss = 0.0f;
     for (int i = tid; i < rank; i += LP_THREADS) ss = fmaf(src[i], src[i], ss);
     ss = block_sum(ss, scratch);
@@ -85,26 +85,28 @@ latent_prepare_kernel(const float* __restrict__ proj, long long ldp, int nh, int
     for (int i = rot + tid; i < dr; i += LP_THREADS) kr[rank + i] = from_f32<TQ>(src[rank + i]);
 }
 
-extern "C" int hb_latent_prepare(const float* proj, long long ldp, int n_heads, int d, int dr, int rank, int down_at,
+// q: the queries' projections [tokens][heads x (d + dr)]; down: [latent | shared key part] per token, needed only with `append`
+// (a layer that reads another layer's latents has none).
+extern "C" int hb_latent_prepare(const float* q, long long ldq_in, const float* down, long long ldd, int n_heads, int d, int dr, int rank,
                                  const float* c_weight, float eps, const float* table, int rot, void* q_out, int q_dtype, long long ldq,
                                  int q_head, int q_rot_at, int q_copy, void* k_cache, void* v_cache, int cache_dtype, const int* page_table, int pt_width, const int* tok_seq,
                                  const int* positions, int n_tokens, int n_pages, int append, int* status, void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && n_heads > 0 && n_heads < 65535 && d > 0 && dr >= 0 && rank > 0, "latent_prepare: bad sizes");
     HB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dr && (rot == 0 || table != nullptr), "latent_prepare: %d rotated dimensions of %d", rot, dr);
-    HB_REQUIRE(ldp >= (long long)down_at + rank + dr && down_at >= n_heads * (d + dr) && ldq >= (long long)n_heads * q_head,
-               "latent_prepare: rows are too short");
+    HB_REQUIRE(ldq_in >= (long long)n_heads * (d + dr) && ldq >= (long long)n_heads * q_head && (!append || (down != nullptr && ldd >= rank + dr && c_weight != nullptr)),
+               "latent_prepare: rows are too short, or there is no latent to append");
     HB_REQUIRE(q_rot_at >= 0 && q_rot_at + dr <= q_head && (q_copy == 0 || (q_copy == d && q_rot_at == d)),
                "latent_prepare: the rotated part at %d of %d columns per head (%d copied) does not fit", q_rot_at, q_head, q_copy);
     HB_REQUIRE(q_dtype == cache_dtype, "latent_prepare: queries and cache must have one dtype");
-    dim3 grid(n_tokens, n_heads + 1);
+    dim3 grid(n_tokens, n_heads + (append ? 1 : 0));
     cudaStream_t s = (cudaStream_t)stream;
     if (q_dtype == HB_BF16)
-        hb_launch(latent_prepare_kernel<bf16>, dim3(grid), dim3(LP_THREADS), 0, s, proj, ldp, n_heads, d, dr, rank, down_at, c_weight, eps,
+        hb_launch(latent_prepare_kernel<bf16>, dim3(grid), dim3(LP_THREADS), 0, s, q, ldq_in, down, ldd, n_heads, d, dr, rank, c_weight, eps,
                   (const float2*)table, rot, (bf16*)q_out, ldq, q_head, q_rot_at, q_copy, (bf16*)k_cache, (bf16*)v_cache, page_table, pt_width, tok_seq, positions,
                   n_pages, append, status);
     else if (q_dtype == HB_F32)
-        hb_launch(latent_prepare_kernel<float>, dim3(grid), dim3(LP_THREADS), 0, s, proj, ldp, n_heads, d, dr, rank, down_at, c_weight, eps,
+        hb_launch(latent_prepare_kernel<float>, dim3(grid), dim3(LP_THREADS), 0, s, q, ldq_in, down, ldd, n_heads, d, dr, rank, c_weight, eps,
                   (const float2*)table, rot, (float*)q_out, ldq, q_head, q_rot_at, q_copy, (float*)k_cache, (float*)v_cache, page_table, pt_width, tok_seq, positions,
                   n_pages, append, status);
     else return hb_fail("latent_prepare: unsupported dtype %d", q_dtype);

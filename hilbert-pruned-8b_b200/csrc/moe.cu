@@ -20,7 +20,12 @@
 //             best runs can be chosen; the `top` largest c among those are the token's experts, their weights s (without
 //             the correction) divided by their sum (+ norm_eps).  Router outputs from `n_real` on are identity experts: they
 //             have no matrices, the plan leaves them out, and moe_combine adds weight * h for them.
-// Experts without a gate (moe_glu with w_up null): act = gelu(W_up h), the exact (erf) form.
+// Experts without a gate (moe_glu, unit 2): act = gelu(W_up h), the exact (erf) form.  Unit 3: act = silu(Wg h) * (Wu h).
+// moe_route with `scoring` 1: the weights are sigmoid(z) of the chosen experts, not divided by anything (the largest z are the
+//             largest sigmoids, so the choice is the same).
+// moe_glu with `in_weights`: an expert is fed weight * h instead of having its result weighted: both products' results are
+//             multiplied by the entry's weight (W (w h) = w (W h)) before the activation, in 32-bit; moe_combine without weights
+//             then adds the experts' results as they are.
 //
 // The products are tiled FP32-pipe kernels (MOE_BM rows x MOE_BN columns x MOE_BK): they serve
 // both precisions, with 32-bit accumulation.  glu_clamp is the same activation for a dense
@@ -44,7 +49,7 @@
 template <typename TH>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restrict__ wr, int* __restrict__ experts,
-                 float* __restrict__ weights, int W, int E, int top) {
+                 float* __restrict__ weights, int W, int E, int top, int scoring) {
     pdl_trigger();
     pdl_wait();
     h = pdl_fresh(h);
@@ -80,7 +85,7 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
             }
             if (best_e >= E) best_e = 0;                  // a row of logits that are not numbers: any expert, the result is not finite anyway
             if (k == 0) zmax = best;
-            const float p = expf(best - zmax);
+            const float p = scoring == 1 ? 1.0f / (1.0f + expf(-best)) : expf(best - zmax);
             denom += p;
             if (lane == 0) {
                 experts[(size_t)t * top + k] = best_e;
@@ -89,22 +94,25 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
             }
             __syncwarp();
         }
-        if (lane == 0)
+        if (lane == 0 && scoring == 0)
             for (int k = 0; k < top; k++) weights[(size_t)t * top + k] /= denom;
     }
 }
 
 extern "C" int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, int* experts, float* weights,
-                            int n_tokens, int width, int n_experts, int top, void* stream) {
+                            int n_tokens, int width, int n_experts, int top, int scoring, void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top >= 1 && top <= n_experts, "moe_route: bad sizes");
+    HB_REQUIRE(scoring == 0 || scoring == 1, "moe_route: scoring %d (0 softmax over the chosen, 1 sigmoid)", scoring);
     const size_t smem = sizeof(float) * ((size_t)width + n_experts);
     HB_REQUIRE(smem <= 48 * 1024, "moe_route: width + experts = %d is too wide", width + n_experts);
     cudaStream_t s = (cudaStream_t)stream;
     if (h_dtype == HB_BF16)
-        hb_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, (const bf16*)h, ldh, w_router, experts, weights, width, n_experts, top);
+        hb_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, (const bf16*)h, ldh, w_router, experts, weights, width, n_experts, top,
+                  scoring);
     else if (h_dtype == HB_F32)
-        hb_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(256), smem, s, (const float*)h, ldh, w_router, experts, weights, width, n_experts, top);
+        hb_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(256), smem, s, (const float*)h, ldh, w_router, experts, weights, width, n_experts, top,
+                  scoring);
     else return hb_fail("moe_route: unsupported dtype %d", h_dtype);
     return hb_check_launch("moe_route");
 }
@@ -278,12 +286,14 @@ extern "C" int hb_moe_max_tiles(int n_entries, int n_experts, int tile_rows) { r
 
 // ------------------------------------------------------------------------------------------------ the experts' products
 __device__ __forceinline__ float moe_gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
-// the first product's epilogue: the clamped gated unit of two matrices (MODE 1), or the exact gelu of one (MODE 2)
+// the first product's epilogue: the clamped gated unit of two matrices (MODE 1), the exact gelu of one (MODE 2), or the plain
+// silu-gated unit of two (MODE 3)
 template <int MODE>
 __device__ __forceinline__ float moe_first_act(float a0, float a1, float limit, float alpha);
 __device__ __forceinline__ float moe_glu(float g, float u, float limit, float alpha);
 template <> __device__ __forceinline__ float moe_first_act<1>(float a0, float a1, float limit, float alpha) { return moe_glu(a0, a1, limit, alpha); }
 template <> __device__ __forceinline__ float moe_first_act<2>(float a0, float a1, float limit, float alpha) { return moe_gelu_erf(a0); }
+template <> __device__ __forceinline__ float moe_first_act<3>(float a0, float a1, float limit, float alpha) { return silu_f32(a0) * a1; }
 template <> __device__ __forceinline__ float moe_first_act<0>(float a0, float a1, float limit, float alpha) { return a0; }
 __device__ __forceinline__ float moe_glu(float g, float u, float limit, float alpha) {
     g = fminf(g, limit);
@@ -297,18 +307,20 @@ template <typename TA, typename TW, typename TO, int MODE>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_product_kernel(const TA* __restrict__ a, long long lda, const TW* __restrict__ w0, const TW* __restrict__ w1,
                    const int* __restrict__ offsets, const int* __restrict__ order, const int* __restrict__ tiles, int top,
-                   TO* __restrict__ out, long long ldo, int N, int K, float limit, float alpha) {
+                   TO* __restrict__ out, long long ldo, int N, int K, float limit, float alpha, const float* __restrict__ in_weights) {
     pdl_trigger();
-    constexpr bool GLU = MODE == 1, FIRST = MODE != 0;        // FIRST: rows gathered by token, results at the slot
+    constexpr bool GLU = MODE == 1 || MODE == 3, FIRST = MODE != 0;        // FIRST: rows gathered by token, results at the slot
     __shared__ float As[MOE_BK][MOE_BM + 1];
     __shared__ float B0[MOE_BK][MOE_BN + 1];
     __shared__ float B1[GLU ? MOE_BK : 1][MOE_BN + 1];
     __shared__ int row_src[MOE_BM], row_dst[MOE_BM];
+    __shared__ float row_w[MOE_BM];
     pdl_wait();
     a = pdl_fresh(a);
     tiles = pdl_fresh(tiles);
     order = pdl_fresh(order);
     offsets = pdl_fresh(offsets);
+    in_weights = pdl_fresh(in_weights);
     if ((int)blockIdx.x >= tiles[0]) return;
     const int e = tiles[1 + 2 * blockIdx.x], r0 = tiles[2 + 2 * blockIdx.x];
     const int rows = min(MOE_BM, offsets[e + 1] - r0);
@@ -318,6 +330,7 @@ moe_product_kernel(const TA* __restrict__ a, long long lda, const TW* __restrict
         const int entry = tid < rows ? order[r0 + tid] : -1;
         row_src[tid] = entry < 0 ? -1 : (FIRST ? entry / top : r0 + tid);
         row_dst[tid] = entry < 0 ? -1 : (FIRST ? r0 + tid : entry);
+        row_w[tid] = (FIRST && in_weights != nullptr && entry >= 0) ? in_weights[entry] : 1.0f;
     }
     __syncthreads();
     const TW* we0 = w0 + (size_t)e * N * K;
@@ -364,7 +377,8 @@ moe_product_kernel(const TA* __restrict__ a, long long lda, const TW* __restrict
         for (int j = 0; j < 2; j++) {
             const int n = n0 + tx * 2 + j;
             if (n >= N) continue;
-            const float v = moe_first_act<MODE>(acc0[i][j], acc1[i][j], limit, alpha);
+            const float rw = row_w[ty * 2 + i];
+            const float v = moe_first_act<MODE>(acc0[i][j] * rw, acc1[i][j] * rw, limit, alpha);
             out[(size_t)dst * ldo + n] = from_f32<TO>(v);
         }
     }
@@ -379,18 +393,20 @@ template <int MODE, typename TO>
 __global__ void __launch_bounds__(MM_THREADS)
 moe_product_mma_kernel(const bf16* __restrict__ a, long long lda, const bf16* __restrict__ w0, const bf16* __restrict__ w1,
                        const int* __restrict__ offsets, const int* __restrict__ order, const int* __restrict__ tiles, int top,
-                       TO* __restrict__ out, long long ldo, int N, int K, float limit, float alpha) {
+                       TO* __restrict__ out, long long ldo, int N, int K, float limit, float alpha, const float* __restrict__ in_weights) {
     pdl_trigger();
     extern __shared__ __align__(128) unsigned char mm_smem[];
-    constexpr bool GLU = MODE == 1, FIRST = MODE != 0;
+    constexpr bool GLU = MODE == 1 || MODE == 3, FIRST = MODE != 0;
     constexpr int TILE_BYTES = MM_BM * MM_BK * 2, MATS = GLU ? 3 : 2, STAGE_BYTES = TILE_BYTES * MATS;
     static_assert(MM_BM == MM_BN && MM_BK * 2 == 128, "one tile shape and 128-byte rows for rows and weights");
     __shared__ int row_src[MM_BM], row_dst[MM_BM];
+    __shared__ float row_w[MM_BM];
     pdl_wait();
     a = pdl_fresh(a);
     tiles = pdl_fresh(tiles);
     order = pdl_fresh(order);
     offsets = pdl_fresh(offsets);
+    in_weights = pdl_fresh(in_weights);
     if ((int)blockIdx.x >= tiles[0]) return;
     const int e = tiles[1 + 2 * blockIdx.x], r0 = tiles[2 + 2 * blockIdx.x];
     const int rows = min(MM_BM, offsets[e + 1] - r0);
@@ -400,6 +416,7 @@ moe_product_mma_kernel(const bf16* __restrict__ a, long long lda, const bf16* __
         const int entry = tid < rows ? order[r0 + tid] : -1;
         row_src[tid] = entry < 0 ? -1 : (FIRST ? entry / top : r0 + tid);
         row_dst[tid] = entry < 0 ? -1 : (FIRST ? r0 + tid : entry);
+        row_w[tid] = (FIRST && in_weights != nullptr && entry >= 0) ? in_weights[entry] : 1.0f;
     }
     __syncthreads();
     const bf16* we0 = w0 + (size_t)e * N * K;
@@ -474,6 +491,7 @@ moe_product_mma_kernel(const bf16* __restrict__ a, long long lda, const bf16* __
 #pragma unroll
     for (int hr = 0; hr < 2; hr++) {
         const int dst = row_dst[wm * 16 + g + 8 * hr];
+        const float rw = row_w[wm * 16 + g + 8 * hr];
         if (dst < 0) continue;
 #pragma unroll
         for (int nt = 0; nt < 4; nt++)
@@ -481,16 +499,17 @@ moe_product_mma_kernel(const bf16* __restrict__ a, long long lda, const bf16* __
             for (int j = 0; j < 2; j++) {
                 const int n = n0 + wn * 32 + nt * 8 + 2 * tg + j;
                 if (n >= N) continue;
-                const float v0 = acc0[nt][2 * hr + j];
-                out[(size_t)dst * ldo + n] = from_f32<TO>(moe_first_act<MODE>(v0, acc1[GLU ? nt : 0][2 * hr + j], limit, alpha));
+                const float v0 = acc0[nt][2 * hr + j] * rw, v1 = acc1[GLU ? nt : 0][2 * hr + j] * rw;
+                out[(size_t)dst * ldo + n] = from_f32<TO>(moe_first_act<MODE>(v0, v1, limit, alpha));
             }
     }
 }
 
 template <int MODE, typename TO>
 static int moe_mma_launch(dim3 grid, cudaStream_t s, const bf16* a, long long lda, const bf16* w0, const bf16* w1, const int* offsets,
-                          const int* order, const int* tiles, int top, TO* out, long long ldo, int N, int K, float limit, float alpha) {
-    constexpr int SMEM = MM_STAGES * MM_BM * MM_BK * 2 * (MODE == 1 ? 3 : 2);
+                          const int* order, const int* tiles, int top, TO* out, long long ldo, int N, int K, float limit, float alpha,
+                          const float* in_weights) {
+    constexpr int SMEM = MM_STAGES * MM_BM * MM_BK * 2 * (MODE == 1 || MODE == 3 ? 3 : 2);
     static bool done[HB_MAX_DEVICES] = {};
     const int slot = hb_device_slot();
     if (!done[slot]) {
@@ -499,15 +518,17 @@ static int moe_mma_launch(dim3 grid, cudaStream_t s, const bf16* a, long long ld
         done[slot] = true;
     }
     hb_launch(moe_product_mma_kernel<MODE, TO>, dim3(grid), dim3(MM_THREADS), SMEM, s, a, lda, w0, w1, offsets, order, tiles, top, out, ldo, N, K,
-              limit, alpha);
+              limit, alpha, in_weights);
     return 0;
 }
 
+// unit 1: the clamped gated unit; 2: the exact gelu of one matrix (passed as w_gate, w_up null); 3: silu(gate) * up.
 extern "C" int hb_moe_glu(const void* h, int h_dtype, long long ldh, const void* w_gate, const void* w_up, int w_dtype, const int* offsets,
                           const int* order, const int* tiles, int max_tiles, int top, void* act, int act_dtype, long long lda, int ff,
-                          int width, float limit, float alpha, int tensor_cores, void* stream) {
+                          int width, int unit, float limit, float alpha, const float* in_weights, int tensor_cores, void* stream) {
     HB_REQUIRE(max_tiles > 0 && ff > 0 && width > 0 && top >= 1, "moe_glu: bad sizes");
     HB_REQUIRE((ff + MOE_BN - 1) / MOE_BN <= 65535, "moe_glu: too many columns");
+    HB_REQUIRE(unit >= 1 && unit <= 3 && (w_up == nullptr) == (unit == 2), "moe_glu: unit %d (1 and 3: two matrices, 2: one)", unit);
     dim3 grid(max_tiles, (ff + MOE_BN - 1) / MOE_BN);
     cudaStream_t s = (cudaStream_t)stream;
     if (tensor_cores) {
@@ -515,31 +536,22 @@ extern "C" int hb_moe_glu(const void* h, int h_dtype, long long ldh, const void*
                    (((uintptr_t)h | (uintptr_t)w_gate | (uintptr_t)w_up) & 15) == 0,   /* a null w_up: one matrix */
                    "moe_glu: the tensor-core variant needs bfloat16 operands with 16-byte aligned rows");
         grid.y = (ff + MM_BN - 1) / MM_BN;
-        if (w_up == nullptr) {
-            if (moe_mma_launch<2, bf16>(grid, s, (const bf16*)h, ldh, (const bf16*)w_gate, (const bf16*)nullptr, offsets, order, tiles, top,
-                                        (bf16*)act, lda, ff, width, limit, alpha)) return 1;
-        } else if (moe_mma_launch<1, bf16>(grid, s, (const bf16*)h, ldh, (const bf16*)w_gate, (const bf16*)w_up, offsets, order, tiles, top,
-                                           (bf16*)act, lda, ff, width, limit, alpha)) return 1;
+#define HB_MG(U)                                                                                                                          \
+    if (moe_mma_launch<U, bf16>(grid, s, (const bf16*)h, ldh, (const bf16*)w_gate, (const bf16*)w_up, offsets, order, tiles, top, (bf16*)act, lda, \
+                                ff, width, limit, alpha, in_weights)) return 1
+        if (unit == 1) { HB_MG(1); } else if (unit == 2) { HB_MG(2); } else { HB_MG(3); }
+#undef HB_MG
         return hb_check_launch("moe_glu");
     }
-    if (w_up == nullptr) {
-        // one matrix per expert (passed as w_gate) and the exact gelu
-        if (h_dtype == HB_BF16 && w_dtype == HB_BF16 && act_dtype == HB_BF16)
-            hb_launch(moe_product_kernel<bf16, bf16, bf16, 2>, dim3(grid), dim3(MOE_THREADS), 0, s, (const bf16*)h, ldh, (const bf16*)w_gate,
-                      (const bf16*)nullptr, offsets, order, tiles, top, (bf16*)act, lda, ff, width, limit, alpha);
-        else if (h_dtype == HB_F32 && w_dtype == HB_F32 && act_dtype == HB_F32)
-            hb_launch(moe_product_kernel<float, float, float, 2>, dim3(grid), dim3(MOE_THREADS), 0, s, (const float*)h, ldh, (const float*)w_gate,
-                      (const float*)nullptr, offsets, order, tiles, top, (float*)act, lda, ff, width, limit, alpha);
-        else return hb_fail("moe_glu: unsupported dtypes h %d w %d act %d", h_dtype, w_dtype, act_dtype);
-        return hb_check_launch("moe_glu");
-    }
-    if (h_dtype == HB_BF16 && w_dtype == HB_BF16 && act_dtype == HB_BF16)
-        hb_launch(moe_product_kernel<bf16, bf16, bf16, 1>, dim3(grid), dim3(MOE_THREADS), 0, s, (const bf16*)h, ldh, (const bf16*)w_gate,
-                  (const bf16*)w_up, offsets, order, tiles, top, (bf16*)act, lda, ff, width, limit, alpha);
-    else if (h_dtype == HB_F32 && w_dtype == HB_F32 && act_dtype == HB_F32)
-        hb_launch(moe_product_kernel<float, float, float, 1>, dim3(grid), dim3(MOE_THREADS), 0, s, (const float*)h, ldh, (const float*)w_gate,
-                  (const float*)w_up, offsets, order, tiles, top, (float*)act, lda, ff, width, limit, alpha);
-    else return hb_fail("moe_glu: unsupported dtypes h %d w %d act %d", h_dtype, w_dtype, act_dtype);
+#define HB_MG(T, U)                                                                                                                       \
+    hb_launch(moe_product_kernel<T, T, T, U>, dim3(grid), dim3(MOE_THREADS), 0, s, (const T*)h, ldh, (const T*)w_gate, (const T*)w_up, offsets,   \
+              order, tiles, top, (T*)act, lda, ff, width, limit, alpha, in_weights)
+    if (h_dtype == HB_BF16 && w_dtype == HB_BF16 && act_dtype == HB_BF16) {
+        if (unit == 1) HB_MG(bf16, 1); else if (unit == 2) HB_MG(bf16, 2); else HB_MG(bf16, 3);
+    } else if (h_dtype == HB_F32 && w_dtype == HB_F32 && act_dtype == HB_F32) {
+        if (unit == 1) HB_MG(float, 1); else if (unit == 2) HB_MG(float, 2); else HB_MG(float, 3);
+    } else return hb_fail("moe_glu: unsupported dtypes h %d w %d act %d", h_dtype, w_dtype, act_dtype);
+#undef HB_MG
     return hb_check_launch("moe_glu");
 }
 
@@ -555,15 +567,17 @@ extern "C" int hb_moe_down(const void* act, int act_dtype, long long lda, const 
                    "moe_down: the tensor-core variant needs bfloat16 operands with 16-byte aligned rows");
         grid.y = (width + MM_BN - 1) / MM_BN;
         if (moe_mma_launch<0, float>(grid, s, (const bf16*)act, lda, (const bf16*)w_down, (const bf16*)nullptr, offsets, order, tiles, top,
-                                         down, ldd, width, ff, 0.0f, 0.0f)) return 1;
+                                         down, ldd, width, ff, 0.0f, 0.0f, (const float*)nullptr)) return 1;
         return hb_check_launch("moe_down");
     }
     if (act_dtype == HB_BF16 && w_dtype == HB_BF16)
         hb_launch(moe_product_kernel<bf16, bf16, float, 0>, dim3(grid), dim3(MOE_THREADS), 0, s, (const bf16*)act, lda, (const bf16*)w_down,
-                  (const bf16*)nullptr, offsets, order, tiles, top, down, ldd, width, ff, 0.0f, 0.0f);
+                  (const bf16*)nullptr, offsets, order, tiles, top, down, ldd, width, ff, 0.0f, 0.0f,
+                  (const float*)nullptr);
     else if (act_dtype == HB_F32 && w_dtype == HB_F32)
         hb_launch(moe_product_kernel<float, float, float, 0>, dim3(grid), dim3(MOE_THREADS), 0, s, (const float*)act, lda, (const float*)w_down,
-                  (const float*)nullptr, offsets, order, tiles, top, down, ldd, width, ff, 0.0f, 0.0f);
+                  (const float*)nullptr, offsets, order, tiles, top, down, ldd, width, ff, 0.0f, 0.0f,
+                  (const float*)nullptr);
     else return hb_fail("moe_down: unsupported dtypes act %d w %d", act_dtype, w_dtype);
     return hb_check_launch("moe_down");
 }
@@ -587,7 +601,7 @@ moe_combine_kernel(const float* __restrict__ down, long long ldd, const float* _
         float v = accumulate ? out[(size_t)t * ldo + c] : 0.0f;
         for (int k = 0; k < top; k++) {
             const bool same = experts != nullptr && experts[(size_t)t * top + k] >= n_real;
-            v = fmaf(weights[(size_t)t * top + k], same ? to_f32(h[(size_t)t * ldh + c]) : down[((size_t)t * top + k) * ldd + c], v);
+            v = fmaf(weights != nullptr ? weights[(size_t)t * top + k] : 1.0f, same ? to_f32(h[(size_t)t * ldh + c]) : down[((size_t)t * top + k) * ldd + c], v);
         }
         out[(size_t)t * ldo + c] = v;
     }

@@ -4,8 +4,9 @@
 // rmsnorm_add: x[t] += y[t] / sqrt(mean(y[t]^2) + eps) * (offset + w); with a second norm
 // (w2, eps2, offset2) the row that was just made is normed again for the next sublayer,
 // h[t] = x[t] / sqrt(mean(x[t]^2) + eps2) * (offset2 + w2), in the same pass: the new residual
-// values stay in registers between the two.  Everything in 32-bit; h in the dtype the next
-// matrix product reads.  One block per token.
+// values stay in registers between the two; with an output h but no second norm (w2 null) h is
+// a copy of the new row.  Everything in 32-bit; h in the dtype the next matrix product reads.
+// One block per token.
 #include "api.h"
 #include "common.cuh"
 
@@ -42,10 +43,14 @@ rmsnorm_add_kernel(const float* __restrict__ y, long long ldy, const float* __re
         ss2 = fmaf(v, v, ss2);
     }
     if (h == nullptr) return;
-    ss2 = block_sum(ss2, scratch);
-    const float r2 = 1.0f / sqrtf(ss2 / (float)n + eps2);
     TO* hr = h + (size_t)t * ldh;
     slot = 0;
+    if (w2 == nullptr) {
+        for (int i = tid; i < n; i += PN_THREADS, slot++) hr[i] = from_f32<TO>(slot < PN_KEEP ? keep[slot] : xr[i]);
+        return;
+    }
+    ss2 = block_sum(ss2, scratch);
+    const float r2 = 1.0f / sqrtf(ss2 / (float)n + eps2);
     for (int i = tid; i < n; i += PN_THREADS, slot++) {
         const float v = slot < PN_KEEP ? keep[slot] : xr[i];       // a thread reads back only what it wrote itself
         hr[i] = from_f32<TO>(v * r2 * (offset2 + w2[i]));
@@ -57,7 +62,7 @@ extern "C" int hb_rmsnorm_add(const float* y, long long ldy, const float* w, flo
                               int n, void* stream) {
     if (n_rows == 0) return 0;
     HB_REQUIRE(n_rows > 0 && n > 0 && ldy >= n && ldx >= n, "rmsnorm_add: bad sizes");
-    HB_REQUIRE(h == nullptr || (w2 != nullptr && ldh >= n), "rmsnorm_add: the second norm needs a weight and an output");
+    HB_REQUIRE(h == nullptr ? w2 == nullptr : ldh >= n, "rmsnorm_add: the second norm needs an output");
     cudaStream_t s = (cudaStream_t)stream;
     if (h == nullptr || h_dtype == HB_F32)
         hb_launch(rmsnorm_add_kernel<float>, dim3(n_rows), dim3(PN_THREADS), 0, s, y, ldy, w, eps, offset, x, ldx, w2, eps2, offset2,

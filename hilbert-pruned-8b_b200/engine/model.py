@@ -132,6 +132,8 @@ class DecoderModel:
         x = ws.buffer("model.x", (cap, H), torch.float32)[:T]
         if getattr(self.embedding, "state_need", None) is not None:
             self.embedding.forward(step.tokens, x, step=step, state=cache.state_view(self.EMBEDDING_STATE))
+        elif getattr(self.embedding, "takes_step", False):
+            self.embedding.forward(step.tokens, x, step=step)      # it leaves something in step.shared for the layers
         else:
             self.embedding.forward(step.tokens, x)
         # Norms at the seam between two blocks may be folded into the products around them: a block

@@ -95,7 +95,7 @@ _SIGNATURES = {
     "hb_layernorm_add": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_float, _c_float, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_ll, _c_ptr, _c_int, _c_ll,
                          _c_int, _c_int, _c_ptr],
     "hb_convert": [_c_ptr, _c_ptr, _c_int, _c_ll, _c_ptr],
-    "hb_latent_prepare": [_c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll,
+    "hb_latent_prepare": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll,
                           _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_latent_gather": [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_latent_scatter": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -106,10 +106,10 @@ _SIGNATURES = {
                     _c_int, _c_ptr],
     "hb_selective_scan": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr,
                           _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_ptr],
-    "hb_moe_route": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr],
+    "hb_moe_route": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
     "hb_moe_plan": [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
     "hb_moe_glu": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ll, _c_int,
-                   _c_int, _c_float, _c_float, _c_int, _c_ptr],
+                   _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_int, _c_ptr],
     "hb_moe_down": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int,
                     _c_ptr],
     "hb_moe_combine": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ptr],
@@ -120,9 +120,13 @@ _SIGNATURES = {
                       _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_ptr],
     "hb_scaled_add_norm": [_c_ptr, _c_ll, _c_float, _c_ptr, _c_ll, _c_ptr, _c_float, _c_float, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr],
     "hb_normed_sum": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_float, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr],
-    "hb_head_scan": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_float,
+    "hb_head_scan": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_float, _c_ptr, _c_float,
                      _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                      _c_ptr, _c_ll, _c_ptr],
+    "hb_group_rmsnorm": [_c_ptr, _c_ll, _c_ptr, _c_float, _c_int, _c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_int, _c_ptr],
+    "hb_gated_sum_norm": [_c_ptr, _c_ll, _c_float, _c_ptr, _c_ll, _c_int, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_float, _c_int, _c_ptr, _c_int, _c_ll,
+                          _c_int, _c_int, _c_ptr],
+    "hb_side_unit": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ll, _c_ll, _c_int, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_glu_clamp": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_float, _c_float, _c_ptr],
 }
 
@@ -1050,22 +1054,26 @@ class Ops:
         self.launches += 1
 
     # ------------------------------------------------------------------ norms on a sublayer's output
-    def rmsnorm_add(self, y, weight, eps: float, offset: float, x, then=None, then_out=None) -> None:
+    def rmsnorm_add(self, y, weight, eps: float, offset: float, x, then=None, then_out=None, copy=None) -> None:
         """``x += y / sqrt(mean(y^2) + eps) * (offset + weight)`` row by row in 32-bit; with ``then = (weight2, eps2,
-        offset2)`` and ``then_out`` also ``then_out = x / sqrt(mean(x^2) + eps2) * (offset2 + weight2)`` of the new rows."""
-        self._dev(y, weight, x, then_out)
+        offset2)`` and ``then_out`` also ``then_out = x / sqrt(mean(x^2) + eps2) * (offset2 + weight2)`` of the new rows; or with
+        ``copy`` (same shape, any kernel dtype) a copy of the new rows there."""
+        self._dev(y, weight, x, then_out, copy)
         T, n = x.shape
-        if y.dtype != torch.float32 or x.dtype != torch.float32 or tuple(y.shape) != (T, n) or (then is None) != (then_out is None):
-            raise KernelError("rmsnorm_add: float32 [tokens, width] input and residual expected")
+        if y.dtype != torch.float32 or x.dtype != torch.float32 or tuple(y.shape) != (T, n) or (then is None) != (then_out is None) \
+                or (copy is not None and then is not None):
+            raise KernelError("rmsnorm_add: float32 [tokens, width] input and residual expected, and a second norm or a copy")
+        if copy is not None:
+            then_out = copy
         w2 = e2 = o2 = None
         if then is not None:
             w2, e2, o2 = then
-            if tuple(then_out.shape) != (T, n):
-                raise KernelError("rmsnorm_add: the second norm's output does not match")
+        if then_out is not None and tuple(then_out.shape) != (T, n):
+            raise KernelError("rmsnorm_add: the second norm's (or the copy's) shape does not match")
         self._call("hb_rmsnorm_add", y.data_ptr(), _rows(y, "rmsnorm_add input"), self._f32_vec(weight, n, "norm weight"), float(eps),
                    float(offset), x.data_ptr(), _rows(x, "residual"), self._f32_vec(w2, n, "norm weight") if then is not None else None,
-                   float(e2 or 0.0), float(o2 or 0.0), then_out.data_ptr() if then is not None else None,
-                   _code(then_out) if then is not None else 0, _rows(then_out, "norm output") if then is not None else 0, T, n,
+                   float(e2 or 0.0), float(o2 or 0.0), then_out.data_ptr() if then_out is not None else None,
+                   _code(then_out) if then_out is not None else 0, _rows(then_out, "norm output") if then_out is not None else 0, T, n,
                    self._stream())
         self.launches += 1
 
@@ -1104,6 +1112,49 @@ class Ops:
         self._call("hb_normed_sum", a.data_ptr(), _rows(a, "first result"), self._f32_vec(wa, n, "norm weight"), b.data_ptr(),
                    _rows(b, "second result"), self._f32_vec(wb, n, "norm weight"), float(eps), out.data_ptr(), _rows(out, "sum"), T, n,
                    1 if accumulate else 0, self._stream())
+        self.launches += 1
+
+    # ------------------------------------------------------------------ norms over parts of a row, gated sums, a token's own input
+    def group_rmsnorm(self, x, weight, eps: float, groups: int, out, rows=None) -> None:
+        """``out[i] = norm(x[r])`` with ``r = rows[i]`` (``rows`` None: every row): every one of ``groups`` runs of equal
+        length is brought to unit mean square by itself (``eps`` inside the root), then ``weight`` scales element by element; 32-bit."""
+        self._dev(x, weight, out, rows)
+        n = x.shape[1]
+        if x.dtype != torch.float32 or out.shape[1] != n or (rows is None and out.shape[0] != x.shape[0]):
+            raise KernelError("group_rmsnorm: float32 [rows, width] input and an output of the same width expected")
+        if rows is not None and (rows.dtype != torch.int32 or rows.numel() != out.shape[0]):
+            raise KernelError("group_rmsnorm: rows must be int32, one per output row")
+        self._call("hb_group_rmsnorm", x.data_ptr(), _rows(x, "group_rmsnorm input"), self._f32_vec(weight, n, "norm weight"), float(eps), int(groups),
+                   out.data_ptr(), _code(out), _rows(out, "group_rmsnorm output"), rows.data_ptr() if rows is not None else None, out.shape[0], n,
+                   self._stream())
+        self.launches += 1
+
+    def gated_sum_norm(self, x, alpha: float, y, weight, eps: float, groups: int, gate=None, gate_bias=None, n_sum: int = 1, copy=None) -> None:
+        """``x = norm(alpha * x + sigmoid(gate + gate_bias) * y)`` row by row in 32-bit, the norm as in ``group_rmsnorm``; ``gate``
+        (float32 ``[tokens, width]``, may be a column range of a wider matrix) None: no gate.  ``n_sum`` > 1: ``y`` holds that many
+        rows per token, which are added first.  ``copy`` (same shape, any kernel dtype) also receives the new rows."""
+        self._dev(x, y, weight, gate, gate_bias, copy)
+        T, n = x.shape
+        if x.dtype != torch.float32 or y.dtype != torch.float32 or n_sum < 1 or tuple(y.shape) != (T * n_sum, n) \
+                or (gate is not None and (gate.dtype != torch.float32 or tuple(gate.shape) != (T, n))) or (copy is not None and tuple(copy.shape) != (T, n)):
+            raise KernelError("gated_sum_norm: float32 residual, result ([tokens * n_sum, width]) and gate logits of one width expected")
+        self._call("hb_gated_sum_norm", x.data_ptr(), _rows(x, "residual"), float(alpha), y.data_ptr(), _rows(y, "sublayer result"), int(n_sum),
+                   gate.data_ptr() if gate is not None else None, _rows(gate, "gate logits") if gate is not None else 0,
+                   self._f32_vec(gate_bias, n, "gate bias") if gate_bias is not None else None, self._f32_vec(weight, n, "norm weight"), float(eps),
+                   int(groups), copy.data_ptr() if copy is not None else None, _code(copy) if copy is not None else 0,
+                   _rows(copy, "residual copy") if copy is not None else 0, T, n, self._stream())
+        self.launches += 1
+
+    def side_unit(self, s, tokens, table, col0: int, out, dim: int) -> None:
+        """``out[t, :dim] = gelu_tanh(s[t, :dim]) * table[tokens[t], col0 : col0 + dim]``, zeros in ``out``'s further columns; ``s``
+        float32, ``table`` row-major ``[vocab, columns]``."""
+        self._dev(s, tokens, table, out)
+        T, n_out = out.shape
+        if s.dtype != torch.float32 or s.shape[0] != T or s.shape[1] < dim or tokens.dtype != torch.int32 or tokens.numel() != T:
+            raise KernelError("side_unit: float32 rows and int32 tokens, one of each per output row, expected")
+        self._call("hb_side_unit", s.data_ptr(), _rows(s, "side_unit input"), tokens.data_ptr(), table.data_ptr(), _code(table),
+                   _rows(table, "side table"), int(col0), table.shape[0], out.data_ptr(), _code(out), _rows(out, "side_unit output"), int(dim), n_out, T,
+                   self.status.data_ptr(), self._stream())
         self.launches += 1
 
     # ------------------------------------------------------------------ window + pooled blocks, sigmoid weights
@@ -1290,27 +1341,32 @@ class Ops:
         self.launches += 1
 
     # ------------------------------------------------------------------ attention over one cached latent per token
-    def latent_prepare(self, proj, heads: int, d: int, dr: int, rank: int, down_at: int, c_weight, eps: float, table, rot: int,
+    def latent_prepare(self, q, down, heads: int, d: int, dr: int, rank: int, c_weight, eps: float, table, rot: int,
                        q_out, cache, step, append: bool, whole_heads: int = 0) -> None:
-        """From a step's float32 projections ``[q (heads x (d + dr)) | ... ]`` with the down projection ``[latent (rank) | shared
-        key part (dr)]`` at column ``down_at``: the latent divided by its root mean square times ``c_weight`` and the key part
+        """From a step's float32 query projections ``q [tokens, heads * (d + dr)]`` and down projection ``down [tokens, rank + dr]`` =
+        ``[latent | shared key part]`` (column ranges of wider matrices are fine; ``down`` and ``c_weight`` may be None without
+        ``append``): the latent divided by its root mean square times ``c_weight`` and the key part
         turned by ``table`` (pairs ``(2i, 2i + 1)`` of its first ``rot`` dimensions) into the cache (key row ``[c | k_r]``, value
         row ``c``); every head's rotated query part turned into ``q_out[t, h, rank:]`` (``q_out`` ``[tokens, heads * (rank + dr)]``).
         With ``whole_heads`` = n: ``q_out`` is ``[tokens, heads * n]`` and receives every head's whole query, ``[unrotated (d) |
         rotated and turned (dr) | zeros]``."""
-        self._dev(proj, c_weight, table, q_out, cache.k, cache.v)
-        T = proj.shape[0]
+        self._dev(q, down, c_weight, table, q_out, cache.k, cache.v)
+        T = q.shape[0]
         q_head = int(whole_heads) if whole_heads else rank + dr
-        if proj.dtype != torch.float32 or tuple(q_out.shape) != (T, heads * q_head) or q_head < (d + dr if whole_heads else 0):
-            raise KernelError("latent_prepare: float32 projections and queries [tokens, heads * (rank + dr)] expected")
+        if q.dtype != torch.float32 or tuple(q.shape) != (T, heads * (d + dr)) or tuple(q_out.shape) != (T, heads * q_head) \
+                or q_head < (d + dr if whole_heads else 0):
+            raise KernelError("latent_prepare: float32 query projections [tokens, heads * (d + dr)] and queries [tokens, heads * (rank + dr)] expected")
+        if append and (down is None or c_weight is None or down.dtype != torch.float32 or tuple(down.shape) != (T, rank + dr)):
+            raise KernelError("latent_prepare: appending needs the float32 down projection [tokens, rank + dr] and the latent's norm weight")
         if rot and (table is None or table.dtype != torch.float32 or not table.is_contiguous() or tuple(table.shape[:2]) != (T, rot // 2)):
             raise KernelError("latent_prepare: rotary table does not match the tokens")
         if tuple(cache.k.shape[1:]) != (1, 64, rank + dr) or tuple(cache.v.shape[1:]) != (1, 64, rank) \
                 or not cache.k.is_contiguous() or not cache.v.is_contiguous() or cache.k.dtype != cache.v.dtype:
             raise KernelError("latent_prepare: cache layer does not match the latent")
         pt = step.page_tables[cache.group]
-        self._call("hb_latent_prepare", proj.data_ptr(), _rows(proj, "projections"), heads, d, dr, rank, int(down_at),
-                   self._f32_vec(c_weight, rank, "latent norm weight"), float(eps), table.data_ptr() if rot else None, int(rot),
+        self._call("hb_latent_prepare", q.data_ptr(), _rows(q, "query projections"), down.data_ptr() if down is not None else None,
+                   _rows(down, "down projection") if down is not None else 0, heads, d, dr, rank,
+                   self._f32_vec(c_weight, rank, "latent norm weight") if c_weight is not None else None, float(eps), table.data_ptr() if rot else None, int(rot),
                    q_out.data_ptr(), _code(q_out), _rows(q_out, "queries"), q_head, d if whole_heads else rank, d if whole_heads else 0,
                    cache.k.data_ptr(), cache.v.data_ptr(), _code(cache.k),
                    pt.data_ptr(), pt.shape[1], step.tok_seq.data_ptr(), step.positions.data_ptr(), T, cache.k.shape[0],
@@ -1423,22 +1479,26 @@ class Ops:
     HEAD_SCAN_CHUNK = 128
 
     def head_scan(self, u, k, q, decay_raw, decay_bias, state, step, out, heads: int, groups: int, head_dim: int, n_state: int,
-                  a_log=None, inv_tau: float = 1.0, skip=None, z=None, q_scale: float = 1.0, workspace=None,
+                  a_log=None, lower=None, q_activation="none", inv_tau: float = 1.0, skip=None, z=None, q_scale: float = 1.0, workspace=None,
                   chunked: Optional[bool] = None) -> None:
         """A recurrent memory per head whose decay depends on the token, over a step's tokens, sequence by sequence:
         ``S <- a S + s u k^T``, ``y = q_scale S^T q + skip u``, ``out = y silu(z)`` (``z`` None: no gate).  ``u`` float32
         ``[tokens, heads * head_dim]``, ``k`` and ``q`` float32 ``[tokens, groups * n_state]`` (heads share them in ``groups``
         runs).  With ``a_log`` (float32 ``[heads]``): ``decay_raw [tokens, heads]`` are step sizes before bias and softplus,
         ``a = exp(-exp(a_log) dt)`` and ``s = dt``.  Without: ``decay_raw [tokens, heads * n_state]``, ``a = sigmoid(decay_raw +
-        decay_bias) ^ inv_tau`` per state index and ``s = 1``.  ``state`` float32 ``[slots, heads * head_dim * n_state]``.
+        decay_bias) ^ inv_tau`` per state index and ``s = 1``.  With ``lower`` (float32 ``[heads * n_state]``; ``k`` None): a forget gate
+        ``a = lower + (1 - lower) sigmoid(decay_raw + decay_bias)`` per state index with ``k = 1 - a`` for a key.
+        ``q_activation`` "silu" is applied to q.  ``state`` float32 ``[slots, heads * head_dim * n_state]``.
         ``chunked`` (default: long portions while heads, channels and sequences are too few to fill the device, given a
         ``workspace``): the tokens of a sequence are cut into chunks that run side by side (three launches)."""
-        self._dev(u, k, q, decay_raw, decay_bias, state, out, a_log, skip, z)
+        self._dev(u, k, q, decay_raw, decay_bias, state, out, a_log, lower, skip, z)
         T = u.shape[0]
-        mode = 0 if a_log is not None else 1
+        mode = 0 if a_log is not None else 2 if lower is not None else 1
+        if (mode == 2) != (k is None):
+            raise KernelError("head_scan: a forget gate takes the place of the keys, the other forms have keys")
         width = heads * head_dim
-        if any(t.dtype != torch.float32 for t in (u, k, q, decay_raw)) or tuple(u.shape) != (T, width) or tuple(out.shape) != (T, width) \
-                or tuple(k.shape) != (T, groups * n_state) or tuple(q.shape) != (T, groups * n_state) \
+        if any(t.dtype != torch.float32 for t in (u, q, decay_raw)) or tuple(u.shape) != (T, width) or tuple(out.shape) != (T, width) \
+                or (k is not None and (k.dtype != torch.float32 or tuple(k.shape) != (T, groups * n_state))) or tuple(q.shape) != (T, groups * n_state) \
                 or tuple(decay_raw.shape) != (T, heads * (n_state if mode else 1)) or (z is not None and (z.dtype != torch.float32 or tuple(z.shape) != (T, width))):
             raise KernelError("head_scan: shapes or dtypes do not agree")
         if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] != width * n_state or state.stride(1) != 1:
@@ -1456,11 +1516,13 @@ class Ops:
             max_chunks = -(-step.max_new // chunk_len)
             carry = workspace.buffer("head_scan.carry", (step.num_seqs * max_chunks * heads * (2 * head_dim * n_state + (n_state if mode else 1)),),
                                      torch.float32)
-        self._call("hb_head_scan", u.data_ptr(), _rows(u, "memory input"), k.data_ptr(), _rows(k, "memory keys"), q.data_ptr(),
+        self._call("hb_head_scan", u.data_ptr(), _rows(u, "memory input"), k.data_ptr() if k is not None else None,
+                   _rows(k, "memory keys") if k is not None else 0, q.data_ptr(),
                    _rows(q, "memory queries"), z.data_ptr() if z is not None else None, _rows(z, "memory gate") if z is not None else 0,
                    decay_raw.data_ptr(), _rows(decay_raw, "decay input"),
                    self._f32_vec(decay_bias, heads * (n_state if mode else 1), "decay bias"),
-                   self._f32_vec(a_log, heads, "A_log") if a_log is not None else None, float(inv_tau),
+                   self._f32_vec(a_log, heads, "A_log") if a_log is not None else None,
+                   self._f32_vec(lower, heads * n_state, "lower bound") if lower is not None else None, self.ACTIVATIONS[q_activation], float(inv_tau),
                    self._f32_vec(skip, heads, "skip weight") if skip is not None else None, float(q_scale), state.data_ptr(),
                    state.stride(0), step.state_slots.data_ptr(), step.seq_start.data_ptr(), out.data_ptr(), _code(out),
                    _rows(out, "memory output"), step.num_seqs, heads, groups, head_dim, n_state, mode, chunk_len, max_chunks,
@@ -1497,9 +1559,12 @@ class Ops:
                    code, -1 if row_gate is None else int(row_gate), self._stream())
         self.launches += 1
 
-    def moe_route(self, h, w_router, top: int, experts, weights) -> None:
+    SCORINGS = {"softmax_chosen": 0, "sigmoid": 1}
+
+    def moe_route(self, h, w_router, top: int, experts, weights, scoring: str = "softmax_chosen") -> None:
         """Per token the ``top`` experts with the largest router logits (``w_router`` float32 ``[experts, width]``, logits in
-        32-bit) into ``experts`` int32 ``[tokens, top]`` and the softmax over those logits into ``weights`` float32."""
+        32-bit) into ``experts`` int32 ``[tokens, top]`` and the softmax over those logits into ``weights`` float32; ``scoring``
+        "sigmoid": the chosen logits' sigmoids instead, not divided by their sum."""
         self._dev(h, w_router, experts, weights)
         T, W = h.shape
         E = w_router.shape[0]
@@ -1508,21 +1573,26 @@ class Ops:
                 or not experts.is_contiguous() or not weights.is_contiguous():
             raise KernelError("moe_route: float32 router [experts, width], int32 and float32 [tokens, top] outputs expected")
         self._call("hb_moe_route", h.data_ptr(), _code(h), _rows(h, "router input"), w_router.data_ptr(), experts.data_ptr(),
-                   weights.data_ptr(), T, W, E, int(top), self._stream())
+                   weights.data_ptr(), T, W, E, int(top), self.SCORINGS[scoring], self._stream())
         self.launches += 1
 
     def moe_max_tiles(self, entries: int, n_experts: int, tile_rows: int) -> int:
         return int(self.lib.hb_moe_max_tiles(int(entries), int(n_experts), int(tile_rows)))
 
     def moe_experts(self, h, experts, weights, w_gate, w_up, w_down, limit: float, alpha: float, out, accumulate: bool, workspace,
-                    cap: int, tag: str = "", identity: bool = False) -> None:
+                    cap: int, tag: str = "", identity: bool = False, unit: str = "clamped_glu", weigh: str = "output"):
         """``out (+)= sum_k weights[t, k] * expert_{experts[t, k]}(h[t])`` with the experts' weights stacked ``[experts, ff,
         width]`` (gate, up) and ``[experts, width, ff]`` (down) in the activations' dtype and the clamped gated unit of
         ``glu_clamp`` between them.  Four launches: plan, gate/up with activation, down, weighted sum.  bfloat16 operands whose
         rows are multiples of 8 elements run the products on the tensor cores (``use_tensor_cores``), all others on the FP32 pipe.
         ``w_up`` None: experts of one matrix, ``act = gelu_erf(w_gate h)`` (``limit`` and ``alpha`` unused).  ``identity``: expert
-        numbers from the stack's size on are identity experts, whose result is ``h[t]`` itself."""
+        numbers from the stack's size on are identity experts, whose result is ``h[t]`` itself.  ``unit`` "silu_glu": ``silu(gate) * up``
+        between the products.  ``weigh`` "input": an expert is fed ``weights[t, k] * h[t]`` and its result is added as it is.
+        ``out`` None: no sum; returns the experts' results, float32 ``[tokens * top, width]`` (engine scratch), for a caller whose
+        own kernel adds a token's rows (``weigh`` "input" only)."""
         self._dev(h, experts, weights, w_gate, w_up, w_down, out)
+        if (out is None and (weigh != "input" or identity)) or weigh not in ("input", "output") or (weigh == "input" and identity):
+            raise KernelError("moe_experts: results are handed on unsummed only when the weights went into the inputs; identity experts weigh outputs")
         T, W = h.shape
         E, F = w_gate.shape[0], w_gate.shape[1]
         top = experts.shape[1]
@@ -1530,7 +1600,7 @@ class Ops:
                 or not (w_gate.is_contiguous() and (w_up is None or w_up.is_contiguous()) and w_down.is_contiguous()) \
                 or not (w_gate.dtype == w_down.dtype == h.dtype) or (w_up is not None and w_up.dtype != h.dtype):
             raise KernelError("moe_experts: stacked contiguous expert weights in the activations' dtype expected")
-        if out.dtype != torch.float32 or tuple(out.shape) != (T, W):
+        if out is not None and (out.dtype != torch.float32 or tuple(out.shape) != (T, W)):
             raise KernelError("moe_experts: float32 [tokens, width] output expected")
         entries = T * top
         most = cap * top
@@ -1547,13 +1617,18 @@ class Ops:
         self._call("hb_moe_glu", h.data_ptr(), _code(h), _rows(h, "expert input"), w_gate.data_ptr(),
                    w_up.data_ptr() if w_up is not None else None, _code(w_gate),
                    offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles, top, act.data_ptr(), _code(act), F, F, W,
-                   float(limit), float(alpha), tc, s)
+                   2 if w_up is None else {"clamped_glu": 1, "silu_glu": 3}[unit], float(limit), float(alpha),
+                   weights.data_ptr() if weigh == "input" else None, tc, s)
         self._call("hb_moe_down", act.data_ptr(), _code(act), F, w_down.data_ptr(), _code(w_down), offsets.data_ptr(), order.data_ptr(),
                    tiles.data_ptr(), max_tiles, top, down.data_ptr(), W, W, F, tc, s)
-        self._call("hb_moe_combine", down.data_ptr(), W, weights.data_ptr(), top, out.data_ptr(), _rows(out, "expert output"), T, W,
+        self.launches += 3
+        if out is None:
+            return down[:entries]
+        self._call("hb_moe_combine", down.data_ptr(), W, weights.data_ptr() if weigh == "output" else None, top, out.data_ptr(), _rows(out, "expert output"), T, W,
                    1 if accumulate else 0, experts.data_ptr() if identity else None, E, h.data_ptr() if identity else None, _code(h),
                    _rows(h, "expert input"), s)
-        self.launches += 4
+        self.launches += 1
+        return None
 
     def glu_clamp(self, gate_up, out, limit: float, alpha: float) -> None:
         """``out = g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` from float32 ``[g | u]``."""

@@ -23,6 +23,8 @@ What a part must provide:
 * position encodings: ``rotation_table(step)`` when the encoding is a rotation of pairs of
   head dimensions by position-dependent angles (the kernels then turn queries and keys
   themselves), else ``apply(q, k, step)`` which turns them in place; see ``PositionEncoding``.
+* residual gates: ``logits(h, step)`` (32-bit, without the bias) and ``bias``.
+* token sides: ``forward(h, x, step, copy=None)``, adding to the 32-bit stream ``x``.
 * blocks (``parts/block.py``): ``ROLES``, ``named_parts()``, ``cache_need()``, ``state_need()``,
   ``forward(x, step, cache, state, append)``.
 * optional, ``folds_norms = True`` on mixers, feed-forwards and blocks: the norms between two
@@ -143,6 +145,13 @@ class Mixer(Part):
     folds_norms = False
     can_overwrite = False
 
+    # ``takes_guest = True``: the mixer's first product can carry further rows for a part that reads the same input (a
+    # residual gate).  The block sets ``guest`` before weights are bound; ``bind`` takes the guest's rows
+    # (``guest.host_rows(dtype)``, None: the guest keeps them) and ``forward`` hands it the columns they gave
+    # (``guest.receive(view)``).
+    takes_guest = False
+    guest = None
+
     def cache_need(self) -> Optional[CacheNeed]:
         return None
 
@@ -154,7 +163,12 @@ class Mixer(Part):
 
 
 class FeedForward(Part):
-    """As ``Mixer``: reads ``h``, adds to ``residual``; ``folds_norms`` and ``can_overwrite`` as there."""
+    """As ``Mixer``: reads ``h``, adds to ``residual``; ``folds_norms`` and ``can_overwrite`` as there.
+
+    ``sums_entries = True`` (may depend on the part's options): ``forward_entries(h, step)`` returns ``(rows, n)``, 32-bit rows
+    ``[tokens * n, width]`` of which n per token add up to the result, for a caller whose own kernel forms that sum."""
+
+    sums_entries = False
 
     folds_norms = False
     can_overwrite = False
@@ -226,6 +240,21 @@ class PositionEncoding(Part):
         raise NotImplementedError(f"{type(self).__name__} gives neither a rotation table nor apply()")
 
 
+def stack_rows(rows: List[torch.Tensor], width: int, guest=None) -> Tuple[torch.Tensor, Optional[int]]:
+    """The matrices ``[n, width]`` one below the other as one product's weight, with zero rows up to a multiple of 8 rows,
+    then the rows of a ``guest`` that lends them (``Mixer.takes_guest``), padded likewise: ``(matrix, first guest row)``,
+    the second None without a guest."""
+    def pad(n):
+        return [torch.zeros(n, width, dtype=rows[0].dtype, device=rows[0].device)] if n else []
+    total = sum(r.shape[0] for r in rows)
+    out, at = list(rows) + pad(-total % 8), None
+    lent = guest.host_rows(rows[0].dtype) if guest is not None else None
+    if lent is not None:
+        at = total + -total % 8
+        out += [lent] + pad(-lent.shape[0] % 8)
+    return torch.cat(out, dim=0).contiguous(), at
+
+
 class Registry:
     def __init__(self, kind: str):
         self.kind = kind
@@ -260,3 +289,5 @@ POSITION_ENCODINGS = Registry("position encoding")
 BLOCKS = Registry("block")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
+RESIDUAL_GATES = Registry("residual gate")
+TOKEN_SIDES = Registry("token side input")

@@ -14,7 +14,8 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, TOKEN_FILTERS, CacheNeed, Registry, StateNeed
+from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, RESIDUAL_GATES, TOKEN_FILTERS, TOKEN_SIDES, CacheNeed, Registry,
+                   StateNeed)
 
 
 class Block:
@@ -352,3 +353,71 @@ class ScaledPreNormBlock(Block):
             self.ff_norm.forward(x, h)
         SandwichBlock._run(self.ff, y, (h, y, step))
         return NORMED if self._add(y, x, ahead) else None
+
+
+@BLOCKS.register("postnorm_sum")
+class PostNormSumBlock(Block):
+    """The norm BEHIND the sum: ``x = norm_a(alpha x + gate_a * mixer(x))``, then, if the layer has a feed-forward, ``x =
+    norm_b(alpha x + gate_b * feed_forward(x))``, then, if the layer has a token side input, ``x += side(x, token)``.  ``alpha`` is the
+    layer's ``block_params["residual_scale"]``; a gate (optional) is one number per element made from what its sublayer reads.
+    The sublayers read the 32-bit stream itself: in 32-bit mode directly, in bfloat16 mode through a rounded copy that the
+    kernel in front leaves while it writes the stream (only a stack's first block converts with a kernel of its own; the
+    protocol across the seam is ``PostNormBlock``'s).  One kernel (``norm_sum`` of the norm) reads a sublayer's 32-bit result,
+    the gate's logits and the stream and writes the stream; the results of a mixture of experts reach it unsummed
+    (``FeedForward.sums_entries``), and the mixer's gate is made by the mixer's own first product where that can take it
+    (``Mixer.takes_guest``)."""
+
+    ROLES = {"mixer_gate": RESIDUAL_GATES, "mixer": MIXERS, "mixer_norm": NORMS, "feed_forward_gate": RESIDUAL_GATES,
+             "feed_forward": FEED_FORWARDS, "feed_forward_norm": NORMS, "token_side": TOKEN_SIDES}
+    OPTIONAL = ("mixer_gate", "feed_forward_gate", "feed_forward", "feed_forward_norm", "token_side")
+    folds_norms = True
+
+    def __init__(self, layer_spec, ctx):
+        super().__init__(layer_spec, ctx)
+        p = self.parts
+        self.mixer, self.mixer_gate, self.mixer_norm = p["mixer"], p.get("mixer_gate"), p["mixer_norm"]
+        self.ff, self.ff_gate, self.ff_norm = p.get("feed_forward"), p.get("feed_forward_gate"), p.get("feed_forward_norm")
+        self.side = p.get("token_side")
+        if (self.ff is None) != (self.ff_norm is None) or (self.ff is None and self.ff_gate is not None):
+            raise ValueError(f"layer {layer_spec.prefix!r}: a feed-forward and its norm come together, and its gate with both")
+        self.alpha = float(layer_spec.block_params.get("residual_scale", 1.0))
+        if self.mixer_gate is not None and getattr(self.mixer, "takes_guest", False) and layer_spec.block_params.get("host_gate", True):
+            self.mixer.guest = self.mixer_gate        # (its role comes first, so its tensors are bound before the mixer's)
+            self.mixer_gate.lends = True
+        self.fuse_entries = True            # tests switch it off to let a mixture of experts sum its results itself
+
+    def _copy_buffer(self, step, size: int):
+        return self.ctx.workspace.buffer("block.h", (self.ctx.max_step_tokens, size), self.ctx.dtype)[:step.num_tokens]
+
+    def fold_request(self, step):
+        size = getattr(self.mixer_norm, "size", None)
+        if self.ctx.dtype == torch.float32 or size is None:
+            return None
+        return StreamCopyAhead((self._copy_buffer(step, size),))
+
+    def _add(self, norm, x, y, gate, h, step, n_sum: int, copy) -> None:
+        logits = gate.logits(h, step) if gate is not None else None
+        norm.norm_sum(x, self.alpha, y, gate=logits, gate_bias=gate.bias if gate is not None else None, n_sum=n_sum, copy=copy)
+
+    def forward(self, x, step, cache, state, append: bool, prepared=None, prepare_next=None):
+        ws, cap, T = self.ctx.workspace, self.ctx.max_step_tokens, step.num_tokens
+        exact = self.ctx.dtype == torch.float32
+        h = x if exact else self._copy_buffer(step, x.shape[1])
+        if not exact and prepared is not COPIED:
+            self.ctx.ops.convert(x, h)
+        y = ws.buffer("block.branch", (cap, x.shape[1]), torch.float32)[:T]
+        ahead = prepare_next[0] if isinstance(prepare_next, StreamCopyAhead) else None
+        inner = None if exact else h                  # the copy that a later sublayer of this layer reads
+        SandwichBlock._run(self.mixer, y, (h, y, step, cache, state, append))
+        self._add(self.mixer_norm, x, y, self.mixer_gate, h, step, 1, inner if self.ff is not None or self.side is not None else ahead)
+        if self.ff is not None:
+            n_sum = 1
+            if self.fuse_entries and getattr(self.ff, "sums_entries", False):
+                rows, n_sum = self.ff.forward_entries(h, step)
+            else:
+                SandwichBlock._run(self.ff, y, (h, y, step))
+                rows = y
+            self._add(self.ff_norm, x, rows, self.ff_gate, h, step, n_sum, inner if self.side is not None else ahead)
+        if self.side is not None:
+            self.side.forward(h, x, step, copy=ahead)
+        return COPIED if ahead is not None else None

@@ -21,12 +21,13 @@ from typing import Dict, List, Optional
 
 import torch
 
-from .base import MIXERS, POSITION_ENCODINGS, Mixer, ParamSpec, StateNeed
+from .base import MIXERS, POSITION_ENCODINGS, Mixer, ParamSpec, StateNeed, stack_rows
 
 
 @MIXERS.register("decay_memory")
 class DecayMemory(Mixer):
     can_overwrite = True
+    takes_guest = True
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -53,8 +54,7 @@ class DecayMemory(Mixer):
             raise ValueError(f"decay_memory: gate {self.gate!r} ('sigmoid' or 'silu')")
         H, d, dv = self.heads, self.d, self.dv
         self.gate_at = 2 * H * d + H * dv
-        self.proj_width = self.gate_at + H * dv
-        self.proj_ld = (self.proj_width + 7) // 8 * 8
+        self.guest_at = None
         self.w_in = self.w_o = self.norm_weight = self.decay = None
 
     def params(self) -> List[ParamSpec]:
@@ -70,10 +70,9 @@ class DecayMemory(Mixer):
         rows = [t["q"], t["k"], t["v"], t["g"]]
         if len({r.dtype for r in rows}) != 1:
             raise ValueError("decay_memory: the input projections are stored in different dtypes")
-        if self.proj_ld > self.proj_width:
-            rows.append(torch.zeros(self.proj_ld - self.proj_width, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
         pack = self.ctx.ops.pack_weight
-        self.w_in = pack(torch.cat(rows, dim=0).contiguous())
+        w_in, self.guest_at = stack_rows(rows, self.hidden, self.guest)
+        self.w_in = pack(w_in)
         self.w_o = pack(t["o"].contiguous())
         self.norm_weight = t["norm"].reshape(-1).to(torch.float32).contiguous() if self.has_norm_weight else None
         self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=rows[0].device)
@@ -87,8 +86,10 @@ class DecayMemory(Mixer):
     def forward(self, h, residual, step, cache, state, append: bool, accumulate: bool = True):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         H, d, dv = self.heads, self.d, self.dv
-        proj = ws.buffer("decay_memory.proj", (cap, self.proj_ld), torch.float32)[:T]
+        proj = ws.buffer("decay_memory.proj", (cap, self.w_in.shape[0]), torch.float32)[:T]
         ops.linear(h, self.w_in, proj)
+        if self.guest_at is not None:
+            self.guest.receive(proj[:, self.guest_at: self.guest_at + self.guest.size])
         o = ws.buffer("decay_memory.o", (cap, H * dv), torch.float32)[:T]
         table, rot = None, 0
         if self.position is not None:

@@ -8,6 +8,9 @@ which carries no decoder prefix (model.c:399-406).
 ``hashed_pair_embedding`` adds an embedding of the pair (previous token, token) to the token's own: row ``(previous *
 mul_prev + token * mul_cur) mod buckets`` of a second table, whose last row (number ``buckets``) serves a sequence's first
 token.  The previous token is per-sequence state (one int32), so that a sequence may be fed in any portions.
+
+``embedding_with_side`` also owns a second table, ``[vocab, columns]``, whose rows are the tokens' own inputs to the layers
+(``parts/token_side.py``); it leaves the table in ``step.shared`` for them.
 """
 from __future__ import annotations
 
@@ -16,6 +19,7 @@ from typing import Dict, List
 import torch
 
 from .base import EMBEDDINGS, HEADS, ParamSpec, Part, StateNeed
+from .token_side import SIDE_TABLE
 
 
 @EMBEDDINGS.register("embedding")
@@ -70,6 +74,29 @@ class HashedPairEmbedding(TokenEmbedding):
         if step is None or state is None:
             raise ValueError("hashed_pair_embedding: the step and the sequences' state are needed (the previous token is state)")
         self.ctx.ops.embed_pair(step, self.weight, self.pairs, state, out, self.buckets, self.mul_prev, self.mul_cur, self.scale)
+
+
+@EMBEDDINGS.register("embedding_with_side")
+class EmbeddingWithSide(TokenEmbedding):
+    takes_step = True           # the model hands the step to forward()
+
+    def __init__(self, spec, ctx):
+        super().__init__(spec, ctx)
+        self.side_columns = int(spec.params["side_columns"])
+        self.side_tensor_name = spec.get("side_tensor_name", "side")
+        self.side = None
+
+    def params(self) -> List[ParamSpec]:
+        return super().params() + [ParamSpec(self.side_tensor_name, (self.vocab, self.side_columns))]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        super().bind(tensors)
+        self.side = tensors[self.side_tensor_name].contiguous()
+
+    def forward(self, tokens, out, step=None) -> None:
+        super().forward(tokens, out)
+        if step is not None:
+            step.shared[SIDE_TABLE] = self.side
 
 
 @HEADS.register("lm_head")

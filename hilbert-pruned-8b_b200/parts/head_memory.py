@@ -14,6 +14,12 @@ per key channel ``alpha = sigmoid(W_a2 (W_a1 h) + a2.b) ^ (1 / tau)``.  Per head
 Each head's o is divided by its root mean square over vdim and multiplied by ``norm`` (size vdim, shared by the heads); the
 heads side by side times ``silu(W_g h)``, then ``W_o``.  State: S, 32-bit, zero at the start.
 
+``forget_gate_memory`` (a gated recurrence whose forget gate doubles as its input gate).  ``q = silu(W_q h)``, ``v = W_v h``
+(heads x dim, heads x vdim) and a forget gate per head and channel ``f = l + (1 - l) sigmoid(W_f h + f.b)`` with a lower bound
+``l`` (tensor ``lower``, heads * dim numbers).  Per head ``S <- diag(f) S + (1 - f) v^T``, ``o = S^T q``: ``1 - f`` stands where
+the other forms have a key.  Each head's o is divided by its root mean square over vdim and multiplied by ``norm`` (size vdim, shared by the
+heads), then ``W_o``.  State: S, 32-bit, zero at the start.
+
 32-bit: the projections' results as the convolution and the recurrence read them, step sizes, decays and their
 logarithms, S, the recurrence's output, gates and norms.  What the output products read is in the activations' dtype.
 """
@@ -23,16 +29,7 @@ from typing import Dict, List, Optional
 
 import torch
 
-from .base import MIXERS, Mixer, ParamSpec, StateNeed
-
-
-def _padded(rows: List[torch.Tensor], width: int, multiple: int = 8) -> torch.Tensor:
-    """The matrices one below the other, with zero rows up to a multiple of ``multiple`` rows."""
-    total = sum(r.shape[0] for r in rows)
-    pad = (-total) % multiple
-    if pad:
-        rows = rows + [torch.zeros(pad, width, dtype=rows[0].dtype, device=rows[0].device)]
-    return torch.cat(rows, dim=0).contiguous()
+from .base import MIXERS, Mixer, ParamSpec, StateNeed, stack_rows
 
 
 @MIXERS.register("state_space_heads")
@@ -71,7 +68,7 @@ class StateSpaceHeads(Mixer):
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         t, pack = tensors, self.ctx.ops.pack_weight
         f32 = lambda x: x.reshape(-1).to(torch.float32).contiguous()
-        self.w_in = pack(_padded([t["in"]], self.hidden))
+        self.w_in = pack(stack_rows([t["in"]], self.hidden)[0])
         self.w_o = pack(t["o"].contiguous())
         self.conv_w = t["conv"].reshape(self.conv_width, self.taps).to(torch.float32).contiguous()
         self.conv_b, self.dt_bias, self.a_log, self.d_skip, self.norm_weight = (f32(t[n]) for n in ("conv.b", "dt_bias", "A_log", "D", "norm"))
@@ -131,7 +128,7 @@ class GatedLinearAttention(Mixer):
         rows = [t["q"], t["k"], t["v"], t["g"], t["a1"]]
         if len({r.dtype for r in rows}) != 1:
             raise ValueError("gated_linear_attention: the input projections are stored in different dtypes")
-        self.w_in = pack(_padded(rows, self.hidden))
+        self.w_in = pack(stack_rows(rows, self.hidden)[0])
         # the decay's second product reads the 32-bit low-rank values where the first product left them (the general product
         # takes a column range of a wider 32-bit matrix; its inner size is the small rank)
         self.w_a2 = t["a2"].contiguous()
@@ -159,3 +156,55 @@ class GatedLinearAttention(Mixer):
         gated = ws.buffer("gated_linear_attention.gated", (cap, H * dv), self.ctx.dtype)[:T]
         ops.gated_norm(o, proj[:, self.g_at: self.g_at + H * dv], self.norm_weight, self.eps, gated, group=dv if H > 1 else None, gate_kind="silu")
         ops.linear(gated, self.w_o, residual, accumulate=accumulate)
+
+
+@MIXERS.register("forget_gate_memory")
+class ForgetGateMemory(Mixer):
+    can_overwrite = True
+    takes_guest = True
+
+    def __init__(self, spec, ctx):
+        super().__init__(spec, ctx)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.heads, self.d, self.dv = int(p["num_heads"]), int(p["head_dim"]), int(p["v_head_dim"])
+        self.eps = float(p["eps"])
+        self.f_at, self.v_at = self.heads * self.d, 2 * self.heads * self.d
+        self.guest_at = None
+        self.w_in = self.w_o = self.f_bias = self.lower = self.norm_weight = None
+
+    def params(self) -> List[ParamSpec]:
+        H, d, dv, W = self.heads, self.d, self.dv, self.hidden
+        return [ParamSpec("q", (H * d, W)), ParamSpec("f", (H * d, W)), ParamSpec("f.b", (H * d,), kind="vector", init="zeros"),
+                ParamSpec("lower", (H * d,), kind="vector", init="zeros"), ParamSpec("v", (H * dv, W)),
+                ParamSpec("norm", (dv,), kind="vector", init="ones"), ParamSpec("o", (W, H * dv))]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        t, pack = tensors, self.ctx.ops.pack_weight
+        rows = [t["q"], t["f"], t["v"]]
+        if len({r.dtype for r in rows}) != 1:
+            raise ValueError("forget_gate_memory: the input projections are stored in different dtypes")
+        w_in, self.guest_at = stack_rows(rows, self.hidden, self.guest)
+        self.w_in, self.w_o = pack(w_in), pack(t["o"].contiguous())
+        self.f_bias, self.lower = (t[n].reshape(-1).to(torch.float32).contiguous() for n in ("f.b", "lower"))
+        self.norm_weight = t["norm"].reshape(-1).to(torch.float32).repeat(self.heads).contiguous()     # one weight for every head
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
+
+    def state_need(self) -> Optional[StateNeed]:
+        return StateNeed((self.heads * self.d * self.dv,), torch.float32)
+
+    def forward(self, h, residual, step, cache, state, append: bool, accumulate: bool = True):
+        ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
+        H, d, dv = self.heads, self.d, self.dv
+        proj = ws.buffer("forget_gate_memory.proj", (cap, self.w_in.shape[0]), torch.float32)[:T]
+        ops.linear(h, self.w_in, proj)
+        if self.guest_at is not None:
+            self.guest.receive(proj[:, self.guest_at: self.guest_at + self.guest.size])
+        o = ws.buffer("forget_gate_memory.o", (cap, H * dv), torch.float32)[:T]
+        ops.head_scan(proj[:, self.v_at: self.v_at + H * dv], None, proj[:, : H * d], proj[:, self.f_at: self.f_at + H * d], self.f_bias,
+                      state, step, o, H, H, dv, d, lower=self.lower, q_activation="silu", workspace=ws)
+        normed = ws.buffer("forget_gate_memory.normed", (cap, H * dv), self.ctx.dtype)[:T]
+        ops.gated_norm(o, None, self.norm_weight, self.eps, normed, group=dv if H > 1 else None)
+        ops.linear(normed, self.w_o, residual, accumulate=accumulate)

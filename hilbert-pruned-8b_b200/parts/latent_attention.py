@@ -7,6 +7,10 @@ are the queries' last ``dr`` dimensions (pairs ``(2i, 2i + 1)`` of the first ``r
 h's unrotated key is ``Wuk_h c`` and its value ``Wuv_h c``; its score for a key is ``(q_u . k_u + q_r . k_r)
 * scale``; causal softmax; the head's result times ``sigmoid(Wg h)_h`` (``head_gate``); output projection.
 
+Options beside that form: ``q_rank``: the queries come through a latent of their own, ``q = Wuq rmsnorm(Wdq h)`` (tensors ``dq``,
+``dq.norm``, ``uq`` in the place of ``q``); ``shares_cache``: the layer has no ``Wdkv`` and reads the latents and key parts that an
+earlier layer of the same rank and rotation cached (its plan entry's ``cache_of``), with its own ``Wuk`` and ``Wuv``.
+
 Only ``c`` and the rotated key part are cached.  The up projections are folded around the attention
 instead of being applied to the cache: with ``q'_h = [Wuk_h^T q_u | q_r]`` the score is ``q'_h . [c | k_r]``
 and the head's result is ``Wuv_h (sum_s p_s c_s)``, which is attention with ONE key/value head whose key row
@@ -26,13 +30,14 @@ from typing import Dict, List
 
 import torch
 
-from .base import MIXERS, POSITION_ENCODINGS, CacheNeed, Mixer, ParamSpec
+from .base import MIXERS, POSITION_ENCODINGS, CacheNeed, Mixer, ParamSpec, stack_rows
 from .sink_attention import softmax_attention
 
 
 @MIXERS.register("latent_attention")
 class LatentAttention(Mixer):
     can_overwrite = True
+    takes_guest = True
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
@@ -51,40 +56,50 @@ class LatentAttention(Mixer):
         self.graph_safe = getattr(self.position, "graph_safe", True)
         H = self.heads
         self.q_width = H * (self.d + self.dr)
-        self.down_at = self.q_width
-        self.gate_at = self.down_at + self.rank + self.dr
-        self.proj_width = self.gate_at + (H if self.head_gate else 0)
-        self.proj_ld = (self.proj_width + 7) // 8 * 8
+        self.q_rank = int(p.get("q_rank") or 0)
+        self.shares_cache = bool(p.get("shares_cache", False))
+        # columns of the input product: [q, or the queries' latent | down projection, if any | gates, if any | a guest's]
+        self.down_at = self.q_rank or self.q_width
+        self.gate_at = self.down_at + (0 if self.shares_cache else self.rank + self.dr)
+        self.guest_at = None
         self.key_dim = self.rank + self.dr
         # head sizes of the written-out form (multiples of 64, as the prompt kernel wants them)
         self.flat_d = (self.d + self.dr + 63) // 64 * 64
         self.flat_dv = (self.dv + 63) // 64 * 64
         self.write_out = True                 # tests switch it off to run every step in the folded form
-        self.w_in = self.w_uk = self.w_uv = self.w_o = self.c_weight = self.w_ukv = self.w_o_flat = None
+        self.w_in = self.w_uk = self.w_uv = self.w_o = self.c_weight = self.w_ukv = self.w_o_flat = self.w_uq = self.q_weight = None
 
     def params(self) -> List[ParamSpec]:
         H, W = self.heads, self.hidden
-        out = [ParamSpec("q", (self.q_width, W)), ParamSpec("dkv", (self.rank + self.dr, W)),
-               ParamSpec("dkv.norm", (self.rank,), kind="vector", init="ones"), ParamSpec("uk", (H * self.d, self.rank)),
-               ParamSpec("uv", (H * self.dv, self.rank)), ParamSpec("o", (W, H * self.dv))]
+        if self.q_rank:
+            out = [ParamSpec("dq", (self.q_rank, W)), ParamSpec("dq.norm", (self.q_rank,), kind="vector", init="ones"),
+                   ParamSpec("uq", (self.q_width, self.q_rank))]
+        else:
+            out = [ParamSpec("q", (self.q_width, W))]
+        if not self.shares_cache:
+            out += [ParamSpec("dkv", (self.rank + self.dr, W)), ParamSpec("dkv.norm", (self.rank,), kind="vector", init="ones")]
+        out += [ParamSpec("uk", (H * self.d, self.rank)), ParamSpec("uv", (H * self.dv, self.rank)), ParamSpec("o", (W, H * self.dv))]
         if self.head_gate:
             out.append(ParamSpec("g", (H, W)))
         return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         t, H = tensors, self.heads
-        rows = [t["q"], t["dkv"]] + ([t["g"]] if self.head_gate else [])
+        rows = [t["dq" if self.q_rank else "q"]] + ([] if self.shares_cache else [t["dkv"]]) + ([t["g"]] if self.head_gate else [])
         if len({r.dtype for r in rows}) != 1:
             raise ValueError("latent_attention: the input projections are stored in different dtypes")
-        if self.proj_ld > self.proj_width:
-            rows.append(torch.zeros(self.proj_ld - self.proj_width, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
         pack = self.ctx.ops.pack_weight
-        self.w_in = pack(torch.cat(rows, dim=0).contiguous())
+        w_in, self.guest_at = stack_rows(rows, self.hidden, self.guest)
+        self.w_in = pack(w_in)
+        if self.q_rank:
+            self.w_uq = pack(t["uq"].contiguous())
+            self.q_weight = t["dq.norm"].reshape(-1).to(torch.float32).contiguous()
         self.w_o = pack(t["o"].contiguous())
         # per head [inputs, outputs]: the key up-projection is stored that way already (it is applied transposed, to the query)
         self.w_uk = t["uk"].reshape(H, self.d, self.rank).contiguous()
         self.w_uv = t["uv"].reshape(H, self.dv, self.rank).transpose(1, 2).contiguous()
-        self.c_weight = t["dkv.norm"].reshape(-1).to(torch.float32).contiguous()
+        if not self.shares_cache:
+            self.c_weight = t["dkv.norm"].reshape(-1).to(torch.float32).contiguous()
         # the written-out form: [Wuk; Wuv] as one matrix, and the output projection with zero columns where values are padded
         self.w_ukv = pack(torch.cat([t["uk"], t["uv"]], dim=0).contiguous())
         if self.flat_dv == self.dv:
@@ -95,7 +110,7 @@ class LatentAttention(Mixer):
             self.w_o_flat = pack(o.reshape(self.hidden, H * self.flat_dv).contiguous())
 
     def weight_bytes(self) -> int:
-        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_uk, self.w_uv, self.w_o))
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_uq, self.w_uk, self.w_uv, self.w_o) if w is not None)
 
     def cache_need(self) -> CacheNeed:
         return CacheNeed(1, self.key_dim, None, v_head_dim=self.rank)
@@ -103,8 +118,19 @@ class LatentAttention(Mixer):
     def forward(self, h, residual, step, cache, state, append: bool, accumulate: bool = True):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         H, d, dr, dv, rank = self.heads, self.d, self.dr, self.dv, self.rank
-        proj = ws.buffer("latent_attention.proj", (cap, self.proj_ld), torch.float32)[:T]
+        if append and self.shares_cache:
+            raise ValueError("latent_attention: a layer without a down projection reads another layer's cache (its plan entry names it)")
+        proj = ws.buffer("latent_attention.proj", (cap, self.w_in.shape[0]), torch.float32)[:T]
         ops.linear(h, self.w_in, proj)
+        if self.guest_at is not None:
+            self.guest.receive(proj[:, self.guest_at: self.guest_at + self.guest.size])
+        q_raw = proj[:, : self.q_width]
+        if self.q_rank:
+            c_q = ws.buffer("latent_attention.c_q", (cap, self.q_rank), self.ctx.dtype)[:T]
+            ops.gated_norm(proj[:, : self.q_rank], None, self.q_weight, self.eps, c_q)
+            q_raw = ws.buffer("latent_attention.q_raw", (cap, self.q_width), torch.float32)[:T]
+            ops.linear(c_q, self.w_uq, q_raw)
+        down = None if self.shares_cache else proj[:, self.down_at: self.down_at + rank + dr]
         table, rot = None, 0
         if self.position is not None and dr:
             rotation = self.position.rotation_table(step)
@@ -113,11 +139,11 @@ class LatentAttention(Mixer):
             table, rot = rotation
         gate = proj[:, self.gate_at: self.gate_at + H] if self.head_gate else None
         if self.written_out(step):
-            self._forward_written_out(proj, table, rot, gate, residual, step, cache, append, accumulate)
+            self._forward_written_out(q_raw, down, table, rot, gate, residual, step, cache, append, accumulate)
             return
         q = ws.buffer("latent_attention.q", (cap, H * self.key_dim), self.ctx.dtype)[:T]
-        ops.latent_prepare(proj, H, d, dr, rank, self.down_at, self.c_weight, self.eps, table, rot, q, cache, step, append)
-        ops.head_linear(proj, d + dr, self.w_uk, q, self.key_dim, d, rank)
+        ops.latent_prepare(q_raw, down, H, d, dr, rank, self.c_weight, self.eps, table, rot, q, cache, step, append)
+        ops.head_linear(q_raw, d + dr, self.w_uk, q, self.key_dim, d, rank)
         mixed = ws.buffer("latent_attention.mixed", (cap, H * rank), torch.float32)[:T]
         softmax_attention(self.ctx, q, H, 1, self.key_dim, rank, cache, step, self.scale, None, 0, mixed)
         attn = ws.buffer("latent_attention.out", (cap, H * dv), self.ctx.dtype)[:T]
@@ -129,11 +155,11 @@ class LatentAttention(Mixer):
         return bool(self.write_out and self.ctx.dtype == torch.bfloat16 and self.ctx.ops.attention_sink_prefill_wanted(
             step, self.heads, self.heads, self.flat_d, self.flat_dv, self.ctx.dtype))
 
-    def _forward_written_out(self, proj, table, rot, gate, residual, step, cache, append: bool, accumulate: bool) -> None:
+    def _forward_written_out(self, q_raw, down, table, rot, gate, residual, step, cache, append: bool, accumulate: bool) -> None:
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         H, d, dr, dv, rank, D, DV = self.heads, self.d, self.dr, self.dv, self.rank, self.flat_d, self.flat_dv
         q = ws.buffer("latent_attention.q_flat", (cap, H * D), torch.bfloat16)[:T]
-        ops.latent_prepare(proj, H, d, dr, rank, self.down_at, self.c_weight, self.eps, table, rot, q, cache, step, append, whole_heads=D)
+        ops.latent_prepare(q_raw, down, H, d, dr, rank, self.c_weight, self.eps, table, rot, q, cache, step, append, whole_heads=D)
         pages = sum((n + 63) // 64 for n in step.host_len)
         width = (step.max_len + 63) // 64
         rows = ws.buffer("latent_attention.flat_c", (pages * 64, rank), torch.bfloat16)

@@ -13,7 +13,10 @@ neighbours (a run's score: its largest choice score; the others count as minus i
 outputs' scores, without the correction, divided by their sum ``+ 1e-20``.  ``identity`` n: the router's last n outputs are
 identity experts, which hand the token's input back (times the weight) and have no tensors.  ``unit`` "gelu": an expert is
 ``W_down gelu(W_up h)`` with the exact (erf) gelu, no gate matrix.  ``shared_gate``: the shared expert's result is multiplied
-by ``sigmoid(W_sg h)``, one number per token (tensor ``shared.sg`` ``[1, width]``).
+by ``sigmoid(W_sg h)``, one number per token (tensor ``shared.sg`` ``[1, width]``).  ``router`` "sigmoid": the ``top`` largest
+logits as in the plain form, weighted by their sigmoids, not divided by anything.  ``unit`` "silu_glu": an expert is
+``W_down (silu(W_gate h) * (W_up h))``.  ``weigh`` "input": an expert is fed ``weight * h`` and its result is added as it is
+(evaluated as ``W (w h) = w (W h)`` in front of the activation, in 32-bit).
 
 Tensors below the part's prefix: ``router``, ``e<i>.gate|up|down``, ``shared.gate|up|down``.  The
 experts' matrices are stacked at load time; the routed products gather their rows on the device
@@ -45,8 +48,11 @@ class MixtureOfExperts(FeedForward):
         self.shared_limit = float(p.get("shared_limit", self.limit))
         self.router = p.get("router", "top_logits")
         self.unit = p.get("unit", "clamped_glu")
-        if self.router not in ("top_logits", "scores") or self.unit not in ("clamped_glu", "gelu"):
-            raise ValueError(f"moe: router {self.router!r} ('top_logits' or 'scores'), unit {self.unit!r} ('clamped_glu' or 'gelu')")
+        self.weigh = p.get("weigh", "output")
+        if self.router not in ("top_logits", "scores", "sigmoid") or self.unit not in ("clamped_glu", "gelu", "silu_glu") \
+                or self.weigh not in ("output", "input"):
+            raise ValueError(f"moe: router {self.router!r} ('top_logits', 'scores' or 'sigmoid'), unit {self.unit!r} ('clamped_glu', 'gelu' or "
+                             f"'silu_glu'), weigh {self.weigh!r} ('output' or 'input')")
         self.identity = int(p.get("identity") or 0)
         self.groups, self.keep = int(p.get("groups") or 1), int(p.get("keep") or 1)
         self.shared_gate = bool(p.get("shared_gate", False))
@@ -57,13 +63,20 @@ class MixtureOfExperts(FeedForward):
             raise ValueError(f"moe: {self.n_outputs} router outputs in {self.groups} groups, {self.keep} kept, top {self.top}")
         if not 1 <= self.top <= self.n_outputs:
             raise ValueError(f"moe: top {self.top} of {self.n_outputs} experts")
+        if self.weigh == "input" and self.identity:
+            raise ValueError("moe: identity experts have their results weighted")
+        if self.unit == "silu_glu" and self.shared_ff:
+            raise ValueError("moe: no shared expert is built for the unit 'silu_glu'")
+        self.glu = self.unit != "gelu"                        # two matrices in front of the activation
+        # the experts' results can be handed on unsummed (one row per token and chosen expert)
+        self.sums_entries = self.weigh == "input" and not self.shared_ff
         self.correction = None
         self.gate_col = None
         self.w_router = self.w_gate = self.w_up = self.w_down = self.ws_gate_up = self.ws_down = None
 
     def params(self) -> List[ParamSpec]:
         W, F = self.hidden, self.ff
-        glu = self.unit == "clamped_glu"
+        glu = self.glu
         out = [ParamSpec("router", (self.n_outputs, W))]
         if self.router == "scores":
             out.append(ParamSpec("correction", (self.n_outputs,), kind="vector", init="zeros"))
@@ -79,7 +92,7 @@ class MixtureOfExperts(FeedForward):
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         t, E = tensors, self.n_experts
         self.w_router = t["router"].to(torch.float32).contiguous()
-        glu = self.unit == "clamped_glu"
+        glu = self.glu
         self.w_gate = torch.stack([t[f"e{e}.gate"] for e in range(E)]).contiguous() if glu else None
         self.w_up = torch.stack([t[f"e{e}.up"] for e in range(E)]).contiguous()
         self.w_down = torch.stack([t[f"e{e}.down"] for e in range(E)]).contiguous()
@@ -104,19 +117,27 @@ class MixtureOfExperts(FeedForward):
         shared = sum(w.numel() * w.element_size() for w in (self.ws_gate_up, self.ws_down)) if self.shared_ff else 0
         return self.w_router.numel() * 4 + self.top * per + shared
 
-    def forward(self, h, residual, step, accumulate: bool = True):
+    def forward_entries(self, h, step):
+        """``(rows, top)``: the chosen experts' results, 32-bit ``[tokens * top, width]``, whose sum per token is the result."""
+        return self._experts(h, step, None, False), self.top
+
+    def _experts(self, h, step, residual, accumulate: bool):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         experts = ws.buffer("moe.experts", (cap, self.top), torch.int32)[:T]
         weights = ws.buffer("moe.weights", (cap, self.top), torch.float32)[:T]
         if self.router == "scores":
             ops.moe_route_scores(h, self.w_router, self.correction, self.top, self.groups, self.keep, experts, weights)
         else:
-            ops.moe_route(h, self.w_router, self.top, experts, weights)
+            ops.moe_route(h, self.w_router, self.top, experts, weights, scoring="sigmoid" if self.router == "sigmoid" else "softmax_chosen")
         if self.unit == "gelu":
-            ops.moe_experts(h, experts, weights, self.w_up, None, self.w_down, 0.0, 0.0, residual, accumulate, ws, cap,
-                            tag=".gelu", identity=self.identity > 0)
-        else:
-            ops.moe_experts(h, experts, weights, self.w_gate, self.w_up, self.w_down, self.limit, self.alpha, residual, accumulate, ws, cap)
+            return ops.moe_experts(h, experts, weights, self.w_up, None, self.w_down, 0.0, 0.0, residual, accumulate, ws, cap,
+                                   tag=".gelu", identity=self.identity > 0, weigh=self.weigh)
+        return ops.moe_experts(h, experts, weights, self.w_gate, self.w_up, self.w_down, self.limit, self.alpha, residual, accumulate, ws, cap,
+                               unit=self.unit, weigh=self.weigh)
+
+    def forward(self, h, residual, step, accumulate: bool = True):
+        ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
+        self._experts(h, step, residual, accumulate)
         if self.shared_ff:
             S = self.shared_ff
             first = self.ws_gate_up.shape[0]

@@ -41,14 +41,14 @@ class RMSNorm(Norm):
     def fold_request(self, out):
         return (self.weight, self.offset, self.eps, out)
 
-    def add_normed(self, y, x, then=None, then_out=None) -> bool:
+    def add_normed(self, y, x, then=None, then_out=None, copy=None) -> bool:
         """``x += norm(y)``; with ``then`` (the RMS norm that reads ``x`` next, or what its ``fold_request`` returned:
         ``(weight, offset, eps, out)``) also ``then(x)`` in the same pass, into ``then_out`` or the request's buffer.
-        Returns whether that output was written."""
+        Returns whether that output was written.  ``copy`` (no ``then``): the stream's new rows in its own dtype as well."""
         second = out2 = None
         if isinstance(then, RMSNorm) and then_out is not None and then.size == self.size:
             second, out2 = (then.weight, then.eps, then.offset), then_out
         elif isinstance(then, tuple) and len(then) == 4 and tuple(then[3].shape) == tuple(x.shape):
             second, out2 = (then[0], then[2], then[1]), then[3]
-        self.ctx.ops.rmsnorm_add(y, self.weight, self.eps, self.offset, x, second, out2)
+        self.ctx.ops.rmsnorm_add(y, self.weight, self.eps, self.offset, x, second, out2, copy=copy)
         return second is not None
