@@ -7,6 +7,7 @@
     python bench.py --design vuladra      # a line of its own: the Vuladra design beside Pogezen layers of equal size
     python bench.py --design tonovik      # a line of its own: the Tonovik design beside Vuladra layers of equal size
     python bench.py --design moponex      # a line of its own: the Moponex design beside Vuladra layers of equal size
+    python bench.py --design ridotar      # a line of its own: the Ridotar design beside Tonovik and Moponex layers of equal size
 
 Prints ONE JSON line.  A step is one decode step of a batch of 8 sequences whose caches hold
 about 8192 tokens each; ``value`` is decoded tokens per second from CUDA events around the
@@ -491,6 +492,30 @@ def moponex_config(z):
             "layers": [dict(ssm, mlp=dense), dict(par, mlp=moe), dict(par, mlp=moe), dict(ssm, mlp=moe)]}
 
 
+# --design ridotar: four Ridotar layers (matrix memory with a fixed decay; forget-gate memory; attention over cached latents
+# with a query latent; the same, reading the layer in front's latents; a mixture of experts and a token side input behind
+# each) beside four Tonovik layers (the closest model: the norm on the sublayers' outputs, the same decayed memory, attention
+# over cached latents of the same sizes) and four Moponex layers (the like of the forget-gate memory and of the mixture of
+# experts), at the same width, heads and head size.  The decayed memory has Tonovik's heads and sizes, the latents Tonovik's
+# ranks with a query latent of three times the key latent's; the forget-gate memory has heads of 128 x 128 numbers; the
+# experts are Moponex's 16 of a quarter of the dense feed-forward's size, two chosen.
+RIDOTAR_GROUPS, RIDOTAR_SIDE = 8, 256
+
+
+def ridotar_config(z):
+    W, hd = z["width"], z["head_dim"]
+    memory = {"type": "lightning", "mixer": {"heads": z["ml_heads"], "dim": z["ml_dim"], "vdim": W // z["ml_heads"],
+                                             "decay": [1.0 - 2.0 ** -(3 + i) for i in range(z["ml_heads"])]}}
+    forget = {"type": "hgrn2", "mixer": {"heads": W // 128, "dim": 128, "vdim": 128}}
+    lat = {"heads": z["heads"], "dim": hd, "rot_dim": hd // 2, "vdim": hd, "q_rank": 12 * hd, "kv_rank": 4 * hd, "scale": (1.5 * hd) ** -0.5,
+           "rot": {"base": 10000.0, "dims": hd // 2}}
+    moe = {"kind": "moe", "router": {"experts": VULADRA_EXPERTS, "top": VULADRA_TOP}, "expert": {"ff": z["ff"] // 4}}
+    return {"architecture": "Ridotar", "norm": {"eps": 1e-6, "groups": RIDOTAR_GROUPS}, "postln_alpha": 1.7, "token_side": {"dim": RIDOTAR_SIDE},
+            "vocab": DESIGN_VOCAB, "width": W,
+            "layers": [dict(memory, mlp=moe), dict(forget, mlp=moe), {"type": "latent_attention", "mixer": lat, "mlp": moe},
+                       {"type": "latent_attention", "mixer": dict(lat, kv_from=2), "mlp": moe}]}
+
+
 def llama_like_config(z):
     return dict(MODEL_8B, hidden_size=z["width"], num_hidden_layers=4, intermediate_size=z["ff"], vocab_size=DESIGN_VOCAB,
                 num_attention_heads=z["heads"], num_key_value_heads=z["kv"], head_dim=z["head_dim"], tie_word_embeddings=True)
@@ -539,7 +564,10 @@ def design_comparison(a) -> int:
     out = {}
     for size, z in DESIGN_SIZES.items():
         row = {}
-        if a.design == "moponex":
+        if a.design == "ridotar":
+            pair = (("ridotar", hb.RidotarConfig.from_dict(ridotar_config(z))), ("tonovik", hb.TonovikConfig.from_dict(tonovik_config(z))),
+                    ("moponex", hb.MoponexConfig.from_dict(moponex_config(z))))
+        elif a.design == "moponex":
             pair = (("moponex", hb.MoponexConfig.from_dict(moponex_config(z))), ("vuladra", hb.VuladraConfig.from_dict(vuladra_config(z))))
         elif a.design == "tonovik":
             pair = (("tonovik", hb.TonovikConfig.from_dict(tonovik_config(z))), ("vuladra", hb.VuladraConfig.from_dict(vuladra_config(z))))
@@ -578,7 +606,7 @@ def design_comparison(a) -> int:
             del llm, eng, seqs
             torch.cuda.empty_cache()
         out[size] = row
-    names = {"moponex": "Moponex layers beside Vuladra layers", "tonovik": "Tonovik layers beside Vuladra layers", "vuladra": "Vuladra layers beside Pogezen layers",
+    names = {"ridotar": "Ridotar layers beside Tonovik and Moponex layers", "moponex": "Moponex layers beside Vuladra layers", "tonovik": "Tonovik layers beside Vuladra layers", "vuladra": "Vuladra layers beside Pogezen layers",
              "pogezen": "Pogezen layers beside Llama layers"}[a.design]
     print(json.dumps({"metric": f"{names} of equal size: prefill of one 2048-token prompt and decode "
                                 f"steps of batch {batch} at context {context}, four layers, random weights",
@@ -683,8 +711,8 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--workload", choices=("8b", "3b", "1b"), default="8b",
                     help="8b: the default line; 3b, 1b: the generation workloads at those shapes (--steps = repeats)")
-    ap.add_argument("--design", choices=("pogezen", "vuladra", "tonovik", "moponex"), default=None,
-                    help="a line of its own: this design's layers beside layers of equal size of the closest other design (prefill, decode, "
+    ap.add_argument("--design", choices=("pogezen", "vuladra", "tonovik", "moponex", "ridotar"), default=None,
+                    help="a line of its own: this design's layers beside layers of equal size of the closest other designs (prefill, decode, "
                          "device time per kernel); the default workload is not run")
     ap.add_argument("--timeline", action="store_true",
                     help="print the per-kernel times of a decode step inside the replayed graph (builds the "
