@@ -116,10 +116,10 @@ class LatentAttention(Mixer):
         return CacheNeed(1, self.key_dim, None, v_head_dim=self.rank)
 
     def forward(self, h, residual, step, cache, state, append: bool, accumulate: bool = True):
-        ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
-        H, d, dr, dv, rank = self.heads, self.d, self.dr, self.dv, self.rank
         if append and self.shares_cache:
             raise ValueError("latent_attention: a layer without a down projection reads another layer's cache (its plan entry names it)")
+        ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
+        H, d, dr, dv, rank = self.heads, self.d, self.dr, self.dv, self.rank
         proj = ws.buffer("latent_attention.proj", (cap, self.w_in.shape[0]), torch.float32)[:T]
         ops.linear(h, self.w_in, proj)
         if self.guest_at is not None:

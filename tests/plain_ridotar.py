@@ -139,7 +139,7 @@ def latent_mixer(h, w: Dict[str, torch.Tensor], c: dict, eps: float, positions, 
     q = (rnd(rms_norm(h @ w["dq"].T, w["dq.norm"], eps)) @ w["uq"].T).reshape(T, H, d + dr)
     q_r = rotate_pairs(q[..., d:], positions, int(rot["dims"]), float(rot["base"]))
     lat, k_r = cached if cached is not None else latents(h, w, c, eps, positions, rnd)
-    k_u, v = (lat @ w["uk"].T).reshape(T, H, d), (lat @ w["uv"].T).reshape(T, H, dv)
+    k_u, v = rnd(lat @ w["uk"].T).reshape(T, H, d), rnd(lat @ w["uv"].T).reshape(T, H, dv)
     qq = torch.cat([rnd(q[..., :d]), rnd(q_r)], dim=-1)
     kk = torch.cat([k_u, k_r[:, None, :].expand(T, H, dr)], dim=-1)
     o = causal_softmax(qq, kk, v, float(c["scale"])).reshape(T, H * dv)
@@ -154,9 +154,20 @@ def route(h, w_router, top: int):
     return best.indices, best.values
 
 
-def moe_ff(h, w: Dict[str, torch.Tensor], c: dict, rnd=same):
-    """The sum of the chosen experts' results, an expert being fed the token's input TIMES its score."""
-    chosen, scores = route(h, w["router"], int(c["router"]["top"]))
+def regret(h, w_router, chosen):
+    """Per token, how far the best router logit left out is above the worst one chosen (negative: the choice is the best)."""
+    z = h @ w_router.T
+    left = z.scatter(1, chosen, -math.inf).max(-1).values
+    return left - torch.gather(z, 1, chosen).min(-1).values
+
+
+def moe_ff(h, w: Dict[str, torch.Tensor], c: dict, rnd=same, chosen=None):
+    """The sum of the chosen experts' results, an expert being fed the token's input TIMES its score.  ``chosen`` [T, top]: a
+    choice made elsewhere (of experts whose logits are nearly tied, say), with the scores of this input."""
+    if chosen is None:
+        chosen, scores = route(h, w["router"], int(c["router"]["top"]))
+    else:
+        scores = torch.gather(torch.sigmoid(h @ w["router"].T), 1, chosen)
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e, s in zip(chosen[t].tolist(), scores[t]):
@@ -196,13 +207,15 @@ class PlainRidotar:
     def _sub(self, prefix: str) -> Dict[str, torch.Tensor]:
         return {n[len(prefix):]: t for n, t in self.w.items() if n.startswith(prefix)}
 
-    def logits(self, tokens: List[int], layers_out: Optional[list] = None):
-        """[T, vocab] for the whole sequence; ``layers_out`` collects the stream after every layer."""
+    def logits(self, tokens: List[int], layers_out: Optional[list] = None, choices: Optional[list] = None, regrets_out: Optional[list] = None):
+        """[T, vocab] for the whole sequence; ``layers_out`` collects the stream after every layer.  ``choices``: per
+        mixture of experts a choice [T, top] to be taken as made, whose ``regret`` ``regrets_out`` collects."""
         c, w, rnd = self.cfg, self.w, self.rnd
         eps, groups, alpha = float(c["norm"]["eps"]), int(c["norm"]["groups"]), float(c["postln_alpha"])
         ids, positions = torch.tensor(tokens), torch.arange(len(tokens))
         x = w["embed"][ids]
         cached = {}
+        made = iter(choices) if choices is not None else None
         for i, layer in enumerate(c["layers"]):
             p, m = f"l{i}.", layer["mixer"]
             mw, h = self._sub(p + "mix."), rnd(x)
@@ -216,7 +229,10 @@ class PlainRidotar:
             x = gated_sum_norm(x, y, h @ w[p + "rg1"].T + w[p + "rg1.b"], alpha, w[p + "norm1"], eps, groups)
             if layer.get("mlp") is not None:
                 h = rnd(x)
-                y = moe_ff(h, self._sub(p + "mlp."), layer["mlp"], rnd)
+                chosen = next(made) if made is not None else None
+                if regrets_out is not None:
+                    regrets_out.append(regret(h, w[p + "mlp.router"], chosen))
+                y = moe_ff(h, self._sub(p + "mlp."), layer["mlp"], rnd, chosen)
                 x = gated_sum_norm(x, y, h @ w[p + "rg2"].T + w[p + "rg2.b"], alpha, w[p + "norm2"], eps, groups)
             if c.get("token_side") is not None:
                 n = int(c["token_side"]["dim"])
