@@ -16,7 +16,8 @@
 
 #define GN_THREADS 256
 #define GN_WARPS (GN_THREADS / 32)
-#define GN_KEEP 4          // vectors of VEC values a thread keeps in registers (rows up to 4096 wide with eight groups or fewer)
+// KEEP: vectors of VEC values a thread keeps in registers between the two (2 or 4, by the run's length: fewer registers, more
+// blocks on an SM); what lies behind them is read again.
 
 template <int VEC> struct gn_vec { float v[VEC]; };
 
@@ -61,7 +62,7 @@ __device__ __forceinline__ void gn_store(bf16* p, const gn_vec<VEC>& r) {
 
 // `load(i)` gives the row's values i .. i + VEC - 1 (it may be called twice for one i, always before that i is stored by the
 // same thread), `store(i, values)` takes the normed and weighted ones.
-template <int VEC, typename Load, typename Store>
+template <int VEC, int KEEP, typename Load, typename Store>
 __device__ __forceinline__ void gn_row(int n, int groups, float eps, const float* __restrict__ w, float* scratch, Load load, Store store) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int size = n / groups;
@@ -73,10 +74,10 @@ __device__ __forceinline__ void gn_row(int n, int groups, float eps, const float
         const int g = team + it * teams;
         const bool on = team < teams && g < groups;
         const int base = g * size;
-        gn_vec<VEC> keep[GN_KEEP];
+        gn_vec<VEC> keep[KEEP];
         float ss = 0.0f;
 #pragma unroll
-        for (int s = 0; s < GN_KEEP; s++) {
+        for (int s = 0; s < KEEP; s++) {
             const int i = first + s * stride;
             if (on && i < size) {
                 keep[s] = load(base + i);
@@ -84,7 +85,7 @@ __device__ __forceinline__ void gn_row(int n, int groups, float eps, const float
                 for (int k = 0; k < VEC; k++) ss = fmaf(keep[s].v[k], keep[s].v[k], ss);
             }
         }
-        for (int i = first + GN_KEEP * stride; on && i < size; i += stride) {
+        for (int i = first + KEEP * stride; on && i < size; i += stride) {
             const gn_vec<VEC> v = load(base + i);
 #pragma unroll
             for (int k = 0; k < VEC; k++) ss = fmaf(v.v[k], v.v[k], ss);
@@ -99,7 +100,7 @@ __device__ __forceinline__ void gn_row(int n, int groups, float eps, const float
         }
         const float r = 1.0f / sqrtf(ss / (float)size + eps);
 #pragma unroll
-        for (int s = 0; s < GN_KEEP; s++) {
+        for (int s = 0; s < KEEP; s++) {
             const int i = first + s * stride;
             if (on && i < size) {
                 const gn_vec<VEC> ww = gn_load<VEC>(w + base + i);
@@ -108,7 +109,7 @@ __device__ __forceinline__ void gn_row(int n, int groups, float eps, const float
                 store(base + i, keep[s]);
             }
         }
-        for (int i = first + GN_KEEP * stride; on && i < size; i += stride) {
+        for (int i = first + KEEP * stride; on && i < size; i += stride) {
             gn_vec<VEC> v = load(base + i);
             const gn_vec<VEC> ww = gn_load<VEC>(w + base + i);
 #pragma unroll
@@ -118,7 +119,7 @@ __device__ __forceinline__ void gn_row(int n, int groups, float eps, const float
     }
 }
 
-template <typename TO, int VEC>
+template <typename TO, int VEC, int KEEP>
 __global__ void __launch_bounds__(GN_THREADS)
 group_rmsnorm_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w, float eps, int groups, TO* __restrict__ out,
                      long long ldo, const int* __restrict__ rows, int n) {
@@ -129,11 +130,11 @@ group_rmsnorm_kernel(const float* __restrict__ x, long long ldx, const float* __
     const int t = blockIdx.x;
     const float* xr = x + (size_t)(rows ? rows[t] : t) * ldx;
     TO* o = out + (size_t)t * ldo;
-    gn_row<VEC>(n, groups, eps, w, scratch, [&](int i) { return gn_load<VEC>(xr + i); }, [&](int i, const gn_vec<VEC>& v) { gn_store<VEC>(o + i, v); });
+    gn_row<VEC, KEEP>(n, groups, eps, w, scratch, [&](int i) { return gn_load<VEC>(xr + i); }, [&](int i, const gn_vec<VEC>& v) { gn_store<VEC>(o + i, v); });
 }
 
-template <typename TC, int VEC>
-__global__ void __launch_bounds__(GN_THREADS)
+template <typename TC, int VEC, int KEEP>
+__global__ void __launch_bounds__(GN_THREADS, KEEP == 2 ? 5 : 4)
 gated_sum_norm_kernel(float* __restrict__ x, long long ldx, float alpha, const float* __restrict__ y, long long ldy, int n_sum,
                       const float* __restrict__ gate, long long ldg, const float* __restrict__ gate_bias, const float* __restrict__ w,
                       float eps, int groups, TC* __restrict__ copy, long long ldc, int n) {
@@ -173,7 +174,13 @@ gated_sum_norm_kernel(float* __restrict__ x, long long ldx, float alpha, const f
         gn_store<VEC>(xr + i, v);
         if (copy != nullptr) gn_store<VEC>(copy + (size_t)t * ldc + i, v);
     };
-    gn_row<VEC>(n, groups, eps, w, scratch, load, store);
+    gn_row<VEC, KEEP>(n, groups, eps, w, scratch, load, store);
+}
+
+// whether two vectors a thread hold a whole run
+static bool gn_short(int n, int groups, int vec) {
+    const int wpg = groups >= GN_WARPS ? 1 : GN_WARPS / groups;
+    return n / groups <= 2 * wpg * 32 * vec;
 }
 
 static bool gn_aligned(const void* p, long long ld, int elem) { return ((uintptr_t)p & (elem * 4 - 1)) == 0 && ld % 4 == 0; }
@@ -186,10 +193,12 @@ extern "C" int hb_group_rmsnorm(const float* x, long long ldx, const float* w, f
     HB_REQUIRE(out_dtype == HB_BF16 || out_dtype == HB_F32, "group_rmsnorm: unsupported output dtype %d", out_dtype);
     const bool vec = (n / groups) % 4 == 0 && gn_aligned(x, ldx, 4) && gn_aligned(w, 4, 4) && gn_aligned(out, ldo, out_dtype == HB_BF16 ? 2 : 4);
     cudaStream_t s = (cudaStream_t)stream;
-#define HB_GN(TO, V) hb_launch(group_rmsnorm_kernel<TO, V>, dim3(n_rows), dim3(GN_THREADS), 0, s, x, ldx, w, eps, groups, (TO*)out, ldo, rows, n)
+#define HB_GN_K(TO, V, K) hb_launch(group_rmsnorm_kernel<TO, V, K>, dim3(n_rows), dim3(GN_THREADS), 0, s, x, ldx, w, eps, groups, (TO*)out, ldo, rows, n)
+#define HB_GN(TO, V) do { if (gn_short(n, groups, V)) HB_GN_K(TO, V, 2); else HB_GN_K(TO, V, 4); } while (0)
     if (out_dtype == HB_BF16) { if (vec) HB_GN(bf16, 4); else HB_GN(bf16, 1); }
     else { if (vec) HB_GN(float, 4); else HB_GN(float, 1); }
 #undef HB_GN
+#undef HB_GN_K
     return hb_check_launch("group_rmsnorm");
 }
 
@@ -205,11 +214,13 @@ extern "C" int hb_gated_sum_norm(float* x, long long ldx, float alpha, const flo
                      (gate == nullptr || gn_aligned(gate, ldg, 4)) && gn_aligned(gate_bias, 4, 4) &&
                      (copy == nullptr || gn_aligned(copy, ldc, copy_dtype == HB_BF16 ? 2 : 4));
     cudaStream_t s = (cudaStream_t)stream;
-#define HB_GS(TC, V)                                                                                                                    \
-    hb_launch(gated_sum_norm_kernel<TC, V>, dim3(n_rows), dim3(GN_THREADS), 0, s, x, ldx, alpha, y, ldy, n_sum, gate, ldg, gate_bias, w, eps, \
+#define HB_GS_K(TC, V, K)                                                                                                               \
+    hb_launch(gated_sum_norm_kernel<TC, V, K>, dim3(n_rows), dim3(GN_THREADS), 0, s, x, ldx, alpha, y, ldy, n_sum, gate, ldg, gate_bias, w, eps, \
               groups, (TC*)copy, ldc, n)
+#define HB_GS(TC, V) do { if (gn_short(n, groups, V)) HB_GS_K(TC, V, 2); else HB_GS_K(TC, V, 4); } while (0)
     if (copy != nullptr && copy_dtype == HB_BF16) { if (vec) HB_GS(bf16, 4); else HB_GS(bf16, 1); }
     else { if (vec) HB_GS(float, 4); else HB_GS(float, 1); }
 #undef HB_GS
+#undef HB_GS_K
     return hb_check_launch("gated_sum_norm");
 }
