@@ -5,11 +5,12 @@ from .vuladra import VuladraConfig
 from .tonovik import TonovikConfig
 from .moponex import MoponexConfig
 from .ridotar import RidotarConfig
+from .mirorax import MiroraxConfig
 from .registry import (config_class_for, load_config, register_architecture, registered_architectures,
                        unregister_architecture)
 from .spec import LayerSpec, ModelSpec, PartSpec, PlanEntry
 
-__all__ = ["ConfigError", "Llama3RopeScaling", "LlamaConfig", "PogezenConfig", "VuladraConfig", "TonovikConfig", "MoponexConfig", "RidotarConfig", "read_config_json", "config_class_for",
+__all__ = ["ConfigError", "Llama3RopeScaling", "LlamaConfig", "PogezenConfig", "VuladraConfig", "TonovikConfig", "MoponexConfig", "RidotarConfig", "MiroraxConfig", "read_config_json", "config_class_for",
            "load_config", "register_architecture", "registered_architectures", "unregister_architecture",
            "LayerSpec", "ModelSpec", "PartSpec", "PlanEntry"]
 
@@ -19,3 +20,4 @@ register_architecture(VuladraConfig)
 register_architecture(TonovikConfig)
 register_architecture(MoponexConfig)
 register_architecture(RidotarConfig)
+register_architecture(MiroraxConfig)

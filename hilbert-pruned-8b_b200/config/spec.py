@@ -81,11 +81,14 @@ class PlanEntry:
     plan more than once.  Cache storage and per-sequence state belong to the plan entry, so
     a layer that runs twice keeps two sets of keys and values.  ``cache_of`` is the index of
     an EARLIER plan entry whose cache this entry reads instead of keeping its own: it then
-    appends nothing.
+    appends nothing.  ``adds`` is the number of a vector of the model's ``stream_vectors`` that is
+    added to every token's stream in front of this entry (what tells the passes over a run of
+    layers apart).
     """
 
     layer: int
     cache_of: Optional[int] = None
+    adds: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -109,6 +112,9 @@ class ModelSpec:
     # the longest sequence the checkpoint was made for (None: not stated); the generation loop
     # ends a request there, the step function does not read it
     max_position: Optional[int] = None
+    # vectors of the stream's width that plan entries add in front of themselves (``PlanEntry.adds``)
+    stream_vectors: Optional[PartSpec] = None
+    stream_vectors_prefix: str = ""
 
     def validate(self) -> None:
         n = len(self.layers)
@@ -117,6 +123,8 @@ class ModelSpec:
         for i, e in enumerate(self.plan):
             if not 0 <= e.layer < n:
                 raise ValueError(f"model spec: plan entry {i} names layer {e.layer} outside 0..{n - 1}")
+            if e.adds is not None and (self.stream_vectors is None or not 0 <= e.adds < int(self.stream_vectors.get("count", 0))):
+                raise ValueError(f"model spec: plan entry {i} adds vector {e.adds}, which the model does not have")
             if e.cache_of is not None:
                 if not 0 <= e.cache_of < i:
                     raise ValueError(

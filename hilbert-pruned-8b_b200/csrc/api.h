@@ -117,7 +117,7 @@ int hb_attention_sink(const void* q, int q_dtype, long long ldq, const void* k_c
                       int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window, int keep_first, int chunk,
                       const float* sink, int all_values, int n_pages, int* status, void* stream);
 int hb_head_mix(const float* partial, const float* mix, void* out, int out_dtype, long long ldo, int n_tokens, int n_heads,
-                int n_kv_heads, int v_dim, int n_val, int ones, const float* gate, long long ldg, void* stream);
+                int n_kv_heads, int v_dim, int n_val, int ones, const float* gate, long long ldg, int gate_per, void* stream);
 // One block per (token, key split) for all heads; see attention_sink.cu.  hb_attention_heads_variant: 0 when the sizes are not built.
 int hb_attention_heads_variant(int n_heads, int n_kv_heads, int head_dim, int v_dim, int cache_dtype, int allow_mma);
 int hb_attention_heads_writes_output(int n_heads, int n_kv_heads, int head_dim, int v_dim, int cache_dtype, int allow_mma);
@@ -127,7 +127,7 @@ int hb_attention_heads(const void* q, int q_dtype, long long ldq, const void* k_
                        int v_dim, float scale, int window, int keep_first, int chunk, const float* sink, int splits, int n_pages,
                        int allow_mma, int* status, void* stream);
 int hb_head_mix_splits(const float* partial, const float* ml, const float* mix, void* out, int out_dtype, long long ldo, int n_tokens,
-                       int n_heads, int n_kv_heads, int v_dim, int splits, int ones, const float* gate, long long ldg, void* stream);
+                       int n_heads, int n_kv_heads, int v_dim, int splits, int ones, const float* gate, long long ldg, int gate_per, void* stream);
 // Flash-style on the tensor cores for steps of many tokens (bfloat16, head sizes 64 or 128); out float32
 // [tokens][heads][n_val][v_dim], n_val = kv heads (every value head) or 1 (the head's own); see attention_sink_prefill.cu.
 int hb_attention_sink_prefill_supported(int n_heads, int n_kv_heads, int head_dim, int v_dim);
@@ -205,10 +205,10 @@ int hb_latent_prepare(const float* q, long long ldq_in, const float* down, long 
                       const float* table, int rot, void* q_out, int q_dtype, long long ldq, int q_head, int q_rot_at, int q_copy, void* k_cache,
                       void* v_cache, int cache_dtype, const int* page_table, int pt_width, const int* tok_seq, const int* positions, int n_tokens,
                       int n_pages, int append, int* status, void* stream);
-int hb_latent_gather(const void* v_cache, const int* page_table, int pt_width, const int* seq_len, int n_seqs, int max_pages, int rank,
-                     void* rows, int* scratch_table, int scratch_width, int n_pages, int* status, void* stream);
-int hb_latent_scatter(const void* kv, long long ldkv, const void* k_cache, const int* page_table, int pt_width, const int* seq_len, int n_seqs,
-                      int max_pages, int n_heads, int d, int dr, int dv, int rank, int hd_out, int vd_out, void* k_out, void* v_out, int n_pages,
+int hb_latent_gather(const void* v_cache, const int* page_table, int pt_width, const int* seq_len, const int* seq_pos0, int window,
+                     int n_seqs, int max_pages, int rank, void* rows, int* scratch_table, int scratch_width, int n_pages, int* status, void* stream);
+int hb_latent_scatter(const void* kv, long long ldkv, const void* k_cache, const int* page_table, int pt_width, const int* seq_len,
+                      const int* seq_pos0, int window, int n_seqs, int max_pages, int n_heads, int d, int dr, int dv, int rank, int hd_out, int vd_out, void* k_out, void* v_out, int n_pages,
                       void* stream);
 int hb_head_linear(const float* in, long long ldi, long long in_head, const void* w, int w_dtype, void* out, int out_dtype, long long ldo,
                    long long out_head, const float* gate, long long ldg, int n_tokens, int n_heads, int n_in, int n_out, void* stream);
@@ -224,8 +224,8 @@ int hb_selective_scan(const void* u, int u_dtype, long long ldu, const float* bc
                       int n_seqs, int inner, int n_state, int chunk_len, int max_chunks, float* carry, long long carry_floats,
                       void* stream);
 // Mixture of experts (moe.cu)
-int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, int* experts, float* weights, int n_tokens, int width,
-                 int n_experts, int top, int scoring, void* stream);
+int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, const float* bias, int* experts, float* weights, int n_tokens,
+                 int width, int n_experts, int top, int scoring, void* stream);
 // tile_rows: hb_moe_tile_rows(tensor_cores), the rows of a plan tile of the products' variant (FP32 pipe, or mma.sync for
 // bfloat16 operands whose rows are multiples of 8 elements)
 int hb_moe_tile_rows(int tensor_cores);
@@ -275,6 +275,11 @@ int hb_group_rmsnorm(const float* x, long long ldx, const float* w, float eps, i
 int hb_gated_sum_norm(float* x, long long ldx, float alpha, const float* y, long long ldy, int n_sum, const float* gate, long long ldg,
                       const float* gate_bias, const float* w, float eps, int groups, void* copy, int copy_dtype, long long ldc, int n_rows, int n,
                       void* stream);
+// x += a * y + b * (z + the weighted sum of n_sum rows of r per token) + v, optionally followed by the next norm of the new rows
+// (parallel_sum.cu): two sublayers side by side, a factor per channel (a, b) on each result, every term optional
+int hb_parallel_sum(float* x, long long ldx, const float* y, long long ldy, const float* a, const float* z, long long ldz, const float* r,
+                    long long ldr, const float* w, int n_sum, const float* b, const float* v, const float* nw, float eps, float offset, void* out,
+                    int out_dtype, long long ldo, int n_rows, int n, void* stream);
 // out = gelu_tanh(s) * table[token][col0 ..], zeros in the columns dim .. n_out (token_side.cu)
 int hb_side_unit(const float* s, long long lds, const int* tokens, const void* table, int table_dtype, long long ldt, long long col0, int vocab,
                  void* out, int out_dtype, long long ldo, int dim, int n_out, int n_tokens, int* status, void* stream);

@@ -274,7 +274,7 @@ extern "C" int hb_attention_sink(const void* q, int q_dtype, long long ldq, cons
 template <typename TO>
 __global__ void __launch_bounds__(256)
 head_mix_kernel(const float* __restrict__ partial, const float* __restrict__ mix, TO* __restrict__ out, long long ldo, int nh,
-                int nkv, int vd, int n_val, int ones, const float* __restrict__ gate, long long ldg) {
+                int nkv, int vd, int n_val, int ones, const float* __restrict__ gate, long long ldg, int gate_per) {
     pdl_trigger();
     pdl_wait();
     partial = pdl_fresh(partial);
@@ -293,24 +293,27 @@ head_mix_kernel(const float* __restrict__ partial, const float* __restrict__ mix
         } else {
             a = pr[(size_t)h * n_val * vd + d];
         }
-        if (gate != nullptr) a *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));     // one gate per (token, head)
+        if (gate != nullptr) a *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + (gate_per > 1 ? e : h)]));   // one per (token, head), or per element
         o[e] = from_f32<TO>(a);
     }
     for (int e = threadIdx.x; e < ones; e += blockDim.x) o[nh * vd + e] = from_f32<TO>(e == 0 ? 1.0f : 0.0f);
 }
 
 extern "C" int hb_head_mix(const float* partial, const float* mix, void* out, int out_dtype, long long ldo, int n_tokens,
-                           int n_heads, int n_kv_heads, int v_dim, int n_val, int ones, const float* gate, long long ldg, void* stream) {
+                           int n_heads, int n_kv_heads, int v_dim, int n_val, int ones, const float* gate, long long ldg, int gate_per,
+                           void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv_heads > 0 && v_dim > 0 && ones >= 0, "head_mix: bad sizes");
     HB_REQUIRE(n_val == 1 || n_val == n_kv_heads, "head_mix: partial results hold %d value heads, 1 or %d expected", n_val, n_kv_heads);
     HB_REQUIRE(mix == nullptr || n_val == n_kv_heads, "head_mix: mixing needs the partial results of every value head");
     HB_REQUIRE(ldo >= (long long)n_heads * v_dim + ones, "head_mix: output rows are too short");
+    HB_REQUIRE(gate == nullptr || ((gate_per == 1 || gate_per == v_dim) && ldg >= (long long)n_heads * gate_per),
+               "head_mix: a gate per (token, head) or per element expected");
     cudaStream_t s = (cudaStream_t)stream;
     if (out_dtype == HB_BF16)
-        hb_launch(head_mix_kernel<bf16>, dim3(n_tokens), dim3(256), 0, s, partial, mix, (bf16*)out, ldo, n_heads, n_kv_heads, v_dim, n_val, ones, gate, ldg);
+        hb_launch(head_mix_kernel<bf16>, dim3(n_tokens), dim3(256), 0, s, partial, mix, (bf16*)out, ldo, n_heads, n_kv_heads, v_dim, n_val, ones, gate, ldg, gate_per);
     else if (out_dtype == HB_F32)
-        hb_launch(head_mix_kernel<float>, dim3(n_tokens), dim3(256), 0, s, partial, mix, (float*)out, ldo, n_heads, n_kv_heads, v_dim, n_val, ones, gate, ldg);
+        hb_launch(head_mix_kernel<float>, dim3(n_tokens), dim3(256), 0, s, partial, mix, (float*)out, ldo, n_heads, n_kv_heads, v_dim, n_val, ones, gate, ldg, gate_per);
     else return hb_fail("head_mix: unsupported output dtype %d", out_dtype);
     return hb_check_launch("head_mix");
 }
@@ -783,7 +786,7 @@ template <typename TO>
 __global__ void __launch_bounds__(256)
 head_mix_splits_kernel(const float* __restrict__ partial, const float* __restrict__ ml, const float* __restrict__ mix,
                        TO* __restrict__ out, long long ldo, int nh, int nkv, int vd, int splits, int ones,
-                       const float* __restrict__ gate, long long ldg) {
+                       const float* __restrict__ gate, long long ldg, int gate_per) {
     // one block per (token, value head c, run of HM_COLS columns of c): first the splits of every head are combined
     // for these columns (shared memory [nh][HM_COLS]), then the heads that use c mix them
     pdl_trigger();
@@ -826,7 +829,7 @@ head_mix_splits_kernel(const float* __restrict__ partial, const float* __restric
         } else {
             a = comb[h * HM_COLS + d];
         }
-        if (gate != nullptr) a *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
+        if (gate != nullptr) a *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + (gate_per > 1 ? h * vd + d_begin + d : h)]));
         o[h * vd + d_begin + d] = from_f32<TO>(a);
     }
     if (c == 0 && blockIdx.z == 0)
@@ -835,18 +838,20 @@ head_mix_splits_kernel(const float* __restrict__ partial, const float* __restric
 
 extern "C" int hb_head_mix_splits(const float* partial, const float* ml, const float* mix, void* out, int out_dtype, long long ldo,
                                   int n_tokens, int n_heads, int n_kv_heads, int v_dim, int splits, int ones, const float* gate,
-                                  long long ldg, void* stream) {
+                                  long long ldg, int gate_per, void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv_heads > 0 && v_dim > 0 && ones >= 0 && splits >= 1, "head_mix: bad sizes");
     HB_REQUIRE(ldo >= (long long)n_heads * v_dim + ones, "head_mix: output rows are too short");
+    HB_REQUIRE(gate == nullptr || ((gate_per == 1 || gate_per == v_dim) && ldg >= (long long)n_heads * gate_per),
+               "head_mix: a gate per (token, head) or per element expected");
     HB_REQUIRE(ml != nullptr || splits == 1, "head_mix: several splits need their maxima and sums");
     const size_t smem = ((size_t)n_heads * splits + (size_t)n_heads * HM_COLS) * sizeof(float);
     HB_REQUIRE(smem <= 48 * 1024 && n_kv_heads <= 65535, "head_mix: too many heads times (splits + value size)");
     cudaStream_t s = (cudaStream_t)stream;
     if (out_dtype == HB_BF16)
-        hb_launch(head_mix_splits_kernel<bf16>, dim3(n_tokens, n_kv_heads, (v_dim + HM_COLS - 1) / HM_COLS), dim3(256), smem, s, partial, ml, mix, (bf16*)out, ldo, n_heads, n_kv_heads, v_dim, splits, ones, gate, ldg);
+        hb_launch(head_mix_splits_kernel<bf16>, dim3(n_tokens, n_kv_heads, (v_dim + HM_COLS - 1) / HM_COLS), dim3(256), smem, s, partial, ml, mix, (bf16*)out, ldo, n_heads, n_kv_heads, v_dim, splits, ones, gate, ldg, gate_per);
     else if (out_dtype == HB_F32)
-        hb_launch(head_mix_splits_kernel<float>, dim3(n_tokens, n_kv_heads, (v_dim + HM_COLS - 1) / HM_COLS), dim3(256), smem, s, partial, ml, mix, (float*)out, ldo, n_heads, n_kv_heads, v_dim, splits, ones, gate, ldg);
+        hb_launch(head_mix_splits_kernel<float>, dim3(n_tokens, n_kv_heads, (v_dim + HM_COLS - 1) / HM_COLS), dim3(256), smem, s, partial, ml, mix, (float*)out, ldo, n_heads, n_kv_heads, v_dim, splits, ones, gate, ldg, gate_per);
     else return hb_fail("head_mix: unsupported output dtype %d", out_dtype);
     return hb_check_launch("head_mix_splits");
 }

@@ -124,25 +124,32 @@ extern "C" int hb_latent_prepare(const float* q, long long ldq_in, const float* 
 // appends the shared rotated key part from the cache and pads keys and values with zeros to the kernel's head sizes.
 #define LE_THREADS 256
 
-__device__ __forceinline__ int le_base_page(const int* __restrict__ seq_len, int b) {
+// With a window only the pages count that the sequence's new tokens can see: from the page of the oldest token on that its
+// first new token (at position seq_pos0) sees.
+__device__ __forceinline__ int le_first_page(const int* __restrict__ seq_pos0, int window, int b) {
+    return hb_oldest_visible(seq_pos0[b], window, 0) / HB_PAGE_TOKENS;
+}
+
+__device__ __forceinline__ int le_base_page(const int* __restrict__ seq_len, const int* __restrict__ seq_pos0, int window, int b) {
     int base = 0;
-    for (int i = 0; i < b; i++) base += (seq_len[i] + HB_PAGE_TOKENS - 1) / HB_PAGE_TOKENS;
+    for (int i = 0; i < b; i++) base += (seq_len[i] + HB_PAGE_TOKENS - 1) / HB_PAGE_TOKENS - le_first_page(seq_pos0, window, i);
     return base;
 }
 
 __global__ void __launch_bounds__(LE_THREADS)
 latent_gather_kernel(const bf16* __restrict__ v_cache, const int* __restrict__ page_table, int pt_width, const int* __restrict__ seq_len,
-                     int rank, bf16* __restrict__ rows, int* __restrict__ scratch_table, int scratch_width, int n_pages, int* status) {
+                     const int* __restrict__ seq_pos0, int window, int rank, bf16* __restrict__ rows, int* __restrict__ scratch_table, int scratch_width, int n_pages, int* status) {
     pdl_trigger();
     pdl_wait();
     v_cache = pdl_fresh(v_cache);
     const int j = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
     const int len = seq_len[b], pages = (len + HB_PAGE_TOKENS - 1) / HB_PAGE_TOKENS;
-    if (j >= pages) {
+    const int first = le_first_page(seq_pos0, window, b);
+    if (j < first || j >= pages) {
         if (tid == 0 && j < scratch_width) scratch_table[(size_t)b * scratch_width + j] = -1;
         return;
     }
-    const int sp = le_base_page(seq_len, b) + j;
+    const int sp = le_base_page(seq_len, seq_pos0, window, b) + j - first;
     if (tid == 0) scratch_table[(size_t)b * scratch_width + j] = sp;
     int page = j < pt_width ? page_table[(size_t)b * pt_width + j] : -1;
     if (page < 0 || page >= n_pages) {
@@ -164,7 +171,7 @@ latent_gather_kernel(const bf16* __restrict__ v_cache, const int* __restrict__ p
 
 __global__ void __launch_bounds__(LE_THREADS)
 latent_scatter_kernel(const bf16* __restrict__ kv, long long ldkv, const bf16* __restrict__ k_cache, const int* __restrict__ page_table,
-                      int pt_width, const int* __restrict__ seq_len, int nh, int d, int dr, int dv, int rank, int hd_out, int vd_out,
+                      int pt_width, const int* __restrict__ seq_len, const int* __restrict__ seq_pos0, int window, int nh, int d, int dr, int dv, int rank, int hd_out, int vd_out,
                       bf16* __restrict__ k_out, bf16* __restrict__ v_out, int n_pages) {
     pdl_trigger();
     pdl_wait();
@@ -172,8 +179,9 @@ latent_scatter_kernel(const bf16* __restrict__ kv, long long ldkv, const bf16* _
     k_cache = pdl_fresh(k_cache);
     const int j = blockIdx.x, b = blockIdx.y, h = blockIdx.z, tid = threadIdx.x;
     const int len = seq_len[b], pages = (len + HB_PAGE_TOKENS - 1) / HB_PAGE_TOKENS;
-    if (j >= pages) return;
-    const int sp = le_base_page(seq_len, b) + j;
+    const int first = le_first_page(seq_pos0, window, b);
+    if (j < first || j >= pages) return;
+    const int sp = le_base_page(seq_len, seq_pos0, window, b) + j - first;
     int page = j < pt_width ? page_table[(size_t)b * pt_width + j] : -1;
     if (page < 0 || page >= n_pages) page = -1;                 // latent_gather has noted it
     const int valid = page < 0 ? 0 : min(HB_PAGE_TOKENS, len - j * HB_PAGE_TOKENS);
@@ -198,26 +206,26 @@ latent_scatter_kernel(const bf16* __restrict__ kv, long long ldkv, const bf16* _
 }
 
 // rows: bfloat16 [scratch pages * 64, rank]; scratch_table int32 [n_seqs, scratch_width]; max_pages: the most pages a sequence has.
-extern "C" int hb_latent_gather(const void* v_cache, const int* page_table, int pt_width, const int* seq_len, int n_seqs, int max_pages,
-                                int rank, void* rows, int* scratch_table, int scratch_width, int n_pages, int* status, void* stream) {
+extern "C" int hb_latent_gather(const void* v_cache, const int* page_table, int pt_width, const int* seq_len, const int* seq_pos0, int window,
+                                int n_seqs, int max_pages, int rank, void* rows, int* scratch_table, int scratch_width, int n_pages, int* status, void* stream) {
     if (n_seqs == 0) return 0;
-    HB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && max_pages > 0 && rank > 0 && scratch_width >= max_pages, "latent_gather: bad sizes");
+    HB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && max_pages > 0 && rank > 0 && window >= 0 && scratch_width >= max_pages, "latent_gather: bad sizes");
     HB_REQUIRE(((uintptr_t)v_cache & 15) == 0 && ((uintptr_t)rows & 15) == 0, "latent_gather: the cache and the rows must be 16-byte aligned");
     hb_launch(latent_gather_kernel, dim3(scratch_width, n_seqs), dim3(LE_THREADS), 0, (cudaStream_t)stream, (const bf16*)v_cache, page_table,
-              pt_width, seq_len, rank, (bf16*)rows, scratch_table, scratch_width, n_pages, status);
+              pt_width, seq_len, seq_pos0, window, rank, (bf16*)rows, scratch_table, scratch_width, n_pages, status);
     return hb_check_launch("latent_gather");
 }
 
 // kv: bfloat16 [scratch pages * 64, ldkv] = [k_u (heads x d) | v (heads x dv) | ...]; k_out [scratch pages, heads, 64, hd_out],
 // v_out [scratch pages, heads, 64, vd_out].
 extern "C" int hb_latent_scatter(const void* kv, long long ldkv, const void* k_cache, const int* page_table, int pt_width, const int* seq_len,
-                                 int n_seqs, int max_pages, int n_heads, int d, int dr, int dv, int rank, int hd_out, int vd_out, void* k_out,
+                                 const int* seq_pos0, int window, int n_seqs, int max_pages, int n_heads, int d, int dr, int dv, int rank, int hd_out, int vd_out, void* k_out,
                                  void* v_out, int n_pages, void* stream) {
     if (n_seqs == 0) return 0;
     HB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && n_heads > 0 && n_heads <= 65535 && max_pages > 0, "latent_scatter: bad sizes");
     HB_REQUIRE(d > 0 && dr >= 0 && dv > 0 && hd_out >= d + dr && vd_out >= dv && ldkv >= (long long)n_heads * (d + dv), "latent_scatter: rows are too short");
     hb_launch(latent_scatter_kernel, dim3(max_pages, n_seqs, n_heads), dim3(LE_THREADS), 0, (cudaStream_t)stream, (const bf16*)kv, ldkv,
-              (const bf16*)k_cache, page_table, pt_width, seq_len, n_heads, d, dr, dv, rank, hd_out, vd_out, (bf16*)k_out, (bf16*)v_out, n_pages);
+              (const bf16*)k_cache, page_table, pt_width, seq_len, seq_pos0, window, n_heads, d, dr, dv, rank, hd_out, vd_out, (bf16*)k_out, (bf16*)v_out, n_pages);
     return hb_check_launch("latent_scatter");
 }
 

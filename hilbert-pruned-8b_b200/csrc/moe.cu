@@ -1,7 +1,7 @@
 // Mixture of experts: router, plan, the experts' products over the tokens routed to them, and
 // the weighted sum.
 //
-// moe_route:  z = Wr h in 32-bit; the `top` largest logits of a token (lowest index on ties) are
+// moe_route:  z = Wr h (+ bias) in 32-bit; the `top` largest logits of a token (lowest index on ties) are
 //             its experts, their weights softmax over those logits alone.
 // moe_plan:   entries (token, k) ordered by expert: offsets[e] .. offsets[e + 1] index `order`, whose
 //             values are entry numbers token * top + k; plus the list of (expert, first row) tiles
@@ -48,8 +48,8 @@
 // ------------------------------------------------------------------------------------------------ route
 template <typename TH>
 __global__ void __launch_bounds__(256)
-moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restrict__ wr, int* __restrict__ experts,
-                 float* __restrict__ weights, int W, int E, int top, int scoring) {
+moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restrict__ wr, const float* __restrict__ bias,
+                 int* __restrict__ experts, float* __restrict__ weights, int W, int E, int top, int scoring) {
     pdl_trigger();
     pdl_wait();
     h = pdl_fresh(h);
@@ -64,7 +64,7 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
         float s = 0.0f;
         for (int i = lane; i < W; i += 32) s = fmaf(w[i], hs[i], s);
         s = warp_sum(s);
-        if (lane == 0) zs[e] = s;
+        if (lane == 0) zs[e] = bias != nullptr ? s + bias[e] : s;
     }
     __syncthreads();
     if (warp == 0) {
@@ -99,7 +99,7 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
     }
 }
 
-extern "C" int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, int* experts, float* weights,
+extern "C" int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, const float* bias, int* experts, float* weights,
                             int n_tokens, int width, int n_experts, int top, int scoring, void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top >= 1 && top <= n_experts, "moe_route: bad sizes");
@@ -108,10 +108,10 @@ extern "C" int hb_moe_route(const void* h, int h_dtype, long long ldh, const flo
     HB_REQUIRE(smem <= 48 * 1024, "moe_route: width + experts = %d is too wide", width + n_experts);
     cudaStream_t s = (cudaStream_t)stream;
     if (h_dtype == HB_BF16)
-        hb_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, (const bf16*)h, ldh, w_router, experts, weights, width, n_experts, top,
+        hb_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, (const bf16*)h, ldh, w_router, bias, experts, weights, width, n_experts, top,
                   scoring);
     else if (h_dtype == HB_F32)
-        hb_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(256), smem, s, (const float*)h, ldh, w_router, experts, weights, width, n_experts, top,
+        hb_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(256), smem, s, (const float*)h, ldh, w_router, bias, experts, weights, width, n_experts, top,
                   scoring);
     else return hb_fail("moe_route: unsupported dtype %d", h_dtype);
     return hb_check_launch("moe_route");

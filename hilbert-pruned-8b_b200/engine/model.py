@@ -13,7 +13,8 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..config.spec import ModelSpec
-from ..parts.base import BLOCKS, EMBEDDINGS, HEADS, NORMS, BuildContext, CacheNeed, ParamSpec, StateNeed
+from ..parts.base import BLOCKS, EMBEDDINGS, HEADS, NORMS, STREAM_VECTORS, BuildContext, CacheNeed, ParamSpec, StateNeed
+from ..parts.block import NORMED, NormAhead
 
 
 class _NullOps:
@@ -37,6 +38,7 @@ class DecoderModel:
         self.blocks = [BLOCKS.get(ls.block)(ls, ctx) for ls in spec.layers]
         self.final_norm = NORMS.build(spec.final_norm, ctx)
         self.head = HEADS.build(spec.head, ctx)
+        self.stream_vectors = STREAM_VECTORS.build(spec.stream_vectors, ctx) if spec.stream_vectors is not None else None
         self.prefix = spec.weight_prefixes[-1]
         self.graph_safe = (all(getattr(part, "graph_safe", True) for _, part in self.named_parts())
                            and all(getattr(b, "graph_safe", True) for b in self.blocks))
@@ -50,6 +52,8 @@ class DecoderModel:
                 out.append((ls.prefix + sub, part))
         out.append((self.spec.final_norm_prefix, self.final_norm))
         out.append((self.spec.head_prefix, self.head))
+        if self.stream_vectors is not None:
+            out.append((self.spec.stream_vectors_prefix, self.stream_vectors))
         return out
 
     def weight_table(self, prefix: Optional[str] = None) -> Dict[str, ParamSpec]:
@@ -110,6 +114,8 @@ class DecoderModel:
             b = self.blocks[e.layer]
             total += sum(p.weight_bytes() for _, p in b.named_parts())
         total += self.final_norm.weight_bytes() + self.head.weight_bytes()
+        if self.stream_vectors is not None:
+            total += self.stream_vectors.weight_bytes()
         return total
 
     def num_parameters(self) -> int:
@@ -124,6 +130,17 @@ class DecoderModel:
         return n
 
     # ------------------------------------------------------------------ forward
+    def _add_vector(self, x, entry, block, step):
+        """Adds the entry's vector to the stream, and in the same pass makes the block's first norm output where its request is
+        of that form; returns what the block then finds prepared."""
+        request = block.fold_request(step) if getattr(block, "folds_norms", False) else None
+        vector = self.stream_vectors.vector(entry.adds)
+        if isinstance(request, NormAhead) and tuple(request[3].shape) == tuple(x.shape):
+            self.ctx.ops.parallel_sum(x, vector=vector, then=(request[0], request[2], request[1]), then_out=request[3])
+            return NORMED
+        self.ctx.ops.parallel_sum(x, vector=vector)
+        return None
+
     def forward(self, step, cache) -> Optional[torch.Tensor]:
         """Runs the step's tokens through the decoder; returns ``[wanted, vocab]`` 32-bit
         logits (None when nothing is wanted)."""
@@ -139,15 +156,26 @@ class DecoderModel:
         # Norms at the seam between two blocks may be folded into the products around them: a block
         # that can says what it needs (fold_request), the block in front prepares it and hands on
         # what it prepared.
-        plan, prepared = self.spec.plan, None
+        # A vector that the next entry adds goes with the request to a block that can add it to its own sum (adds_vector).
+        plan, prepared, added = self.spec.plan, None, False
         for i, e in enumerate(plan):
             owner = i if e.cache_of is None else e.cache_of
             block = self.blocks[e.layer]
+            if e.adds is not None and not added:
+                prepared = self._add_vector(x, e, block, step)
             args = (x, step, cache.view(owner), cache.state_view(i), e.cache_of is None)
+            after = plan[i + 1] if i + 1 < len(plan) else None
+            added = False
             if getattr(block, "folds_norms", False):
-                nxt = self.blocks[plan[i + 1].layer] if i + 1 < len(plan) else None
+                nxt = self.blocks[after.layer] if after is not None else None
                 request = nxt.fold_request(step) if nxt is not None and getattr(nxt, "folds_norms", False) else None
-                prepared = block.forward(*args, prepared=prepared, prepare_next=request)
+                kw = {}
+                if after is not None and after.adds is not None:
+                    if getattr(block, "adds_vector", False):
+                        kw["vector"], added = self.stream_vectors.vector(after.adds), True
+                    else:
+                        request = None              # the norm in front of the next entry reads the stream behind the vector
+                prepared = block.forward(*args, prepared=prepared, prepare_next=request, **kw)
             else:
                 block.forward(*args)
                 prepared = None

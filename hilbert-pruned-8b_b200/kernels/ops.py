@@ -38,13 +38,13 @@ _SIGNATURES = {
                        _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_attention_sink": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
                           _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr],
-    "hb_head_mix": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_ptr],
+    "hb_head_mix": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_ptr],
     "hb_attention_heads": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                            _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int,
                            _c_int, _c_ptr, _c_ptr],
     "hb_attention_sink_prefill": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                                   _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
-    "hb_head_mix_splits": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_ptr],
+    "hb_head_mix_splits": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_ptr],
     "hb_mlstm_scan": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_float, _c_float, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
                       _c_int, _c_int, _c_ptr],
     "hb_mlstm_chunks": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_float, _c_float, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
@@ -97,8 +97,8 @@ _SIGNATURES = {
     "hb_convert": [_c_ptr, _c_ptr, _c_int, _c_ll, _c_ptr],
     "hb_latent_prepare": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll,
                           _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
-    "hb_latent_gather": [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr],
-    "hb_latent_scatter": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+    "hb_latent_gather": [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr],
+    "hb_latent_scatter": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                           _c_ptr, _c_ptr, _c_int, _c_ptr],
     "hb_head_linear": [_c_ptr, _c_ll, _c_ll, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int,
                        _c_ptr],
@@ -106,7 +106,7 @@ _SIGNATURES = {
                     _c_int, _c_ptr],
     "hb_selective_scan": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr,
                           _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_ptr],
-    "hb_moe_route": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
+    "hb_moe_route": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
     "hb_moe_plan": [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
     "hb_moe_glu": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ll, _c_int,
                    _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_int, _c_ptr],
@@ -126,6 +126,8 @@ _SIGNATURES = {
     "hb_group_rmsnorm": [_c_ptr, _c_ll, _c_ptr, _c_float, _c_int, _c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_int, _c_ptr],
     "hb_gated_sum_norm": [_c_ptr, _c_ll, _c_float, _c_ptr, _c_ll, _c_int, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_float, _c_int, _c_ptr, _c_int, _c_ll,
                           _c_int, _c_int, _c_ptr],
+    "hb_parallel_sum": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_float,
+                        _c_float, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr],
     "hb_side_unit": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ll, _c_ll, _c_int, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_glu_clamp": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_float, _c_float, _c_ptr],
 }
@@ -604,17 +606,25 @@ class Ops:
             raise KernelError("head gate: float32 [tokens, heads] expected")
         return gate.data_ptr(), _rows(gate, "head gate")
 
+    def _result_gate(self, gate, T: int, heads: int, v_dim: int):
+        """Pointer, row stride and columns per head (1 or ``v_dim``) of a gate on the heads' results: float32 with contiguous rows,
+        one number per token and head (``[tokens, heads]``) or one per element (``[tokens, heads * v_dim]``)."""
+        if gate is not None and v_dim > 1 and tuple(gate.shape) == (T, heads * v_dim):
+            return (*self._head_gate(gate, T, heads * v_dim), v_dim)
+        return (*self._head_gate(gate, T, heads), 1)
+
     def head_mix(self, partial, mix, out, heads: int, kv_heads: int, v_dim: int, n_val: int, ones: int = 0, gate=None) -> None:
         """``out[t, h] = sum_g mix[h, g] partial[t, g, kv(h)]`` (``mix`` None: the head's own); ``ones`` more columns
         (a one, then zeros) follow, through which the next product adds a bias stored as a column of its weight.  ``gate``
-        float32 ``[tokens, heads]``: head h's result is multiplied by ``sigmoid(gate[t, h])``."""
+        float32 ``[tokens, heads]``: head h's result is multiplied by ``sigmoid(gate[t, h])``; or ``[tokens, heads * v_dim]``: every
+        element by its own."""
         self._dev(partial, mix, out, gate)
         T = out.shape[0]
         if out.shape[1] != heads * v_dim + ones or partial.numel() != T * heads * n_val * v_dim:
             raise KernelError("head_mix: shapes do not agree")
         self._call("hb_head_mix", partial.data_ptr(), self._f32_vec(mix, heads * heads, "head mix") if mix is not None else None,
                    out.data_ptr(), _code(out), _rows(out, "head_mix output"), T, heads, kv_heads, v_dim, n_val, ones,
-                   *self._head_gate(gate, T, heads), self._stream())
+                   *self._result_gate(gate, T, heads, v_dim), self._stream())
         self.launches += 1
 
     SINK_PREFILL_FROM = 16          # steps whose longest portion has at least so many tokens run the flash-style kernel
@@ -709,7 +719,7 @@ class Ops:
             raise KernelError("head_mix_splits: shapes do not agree")
         self._call("hb_head_mix_splits", partial.data_ptr(), ml.data_ptr() if ml is not None else None,
                    self._f32_vec(mix, heads * heads, "head mix") if mix is not None else None, out.data_ptr(), _code(out),
-                   _rows(out, "head_mix output"), T, heads, kv_heads, v_dim, splits, ones, *self._head_gate(gate, T, heads), self._stream())
+                   _rows(out, "head_mix output"), T, heads, kv_heads, v_dim, splits, ones, *self._result_gate(gate, T, heads, v_dim), self._stream())
         self.launches += 1
 
     # ------------------------------------------------------------------ matrix memory (mLSTM)
@@ -1145,6 +1155,33 @@ class Ops:
                    _rows(copy, "residual copy") if copy is not None else 0, T, n, self._stream())
         self.launches += 1
 
+    def parallel_sum(self, x, y=None, a=None, z=None, entries=None, entry_weights=None, n_sum: int = 0, b=None, vector=None, then=None,
+                     then_out=None) -> None:
+        """``x += a * y + b * (z + sum_k entry_weights[t, k] * entries[t * n_sum + k]) + vector`` row by row in 32-bit, every term
+        optional: ``y``, ``z`` float32 ``[tokens, width]``, ``entries`` float32 ``[tokens * n_sum, width]`` (``entry_weights`` float32 ``[tokens,
+        n_sum]``, None: ones), ``a``, ``b``, ``vector`` float32 ``[width]``.  With ``then = (weight, eps, offset)`` and ``then_out`` also
+        ``then_out = x / sqrt(mean(x^2) + eps) * (offset + weight)`` of the new rows, in the same pass."""
+        self._dev(x, y, a, z, entries, entry_weights, b, vector, then_out)
+        T, n = x.shape
+        n_sum = int(n_sum) if entries is not None else 0
+        for t, rows, what in ((x, T, "residual"), (y, T, "first result"), (z, T, "second result"), (entries, T * n_sum, "entries")):
+            if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != (rows, n)):
+                raise KernelError(f"parallel_sum: float32 [{rows}, {n}] expected for the {what}")
+        if entry_weights is not None and (entry_weights.dtype != torch.float32 or not entry_weights.is_contiguous()
+                                          or tuple(entry_weights.shape) != (T, n_sum)):
+            raise KernelError("parallel_sum: contiguous float32 weights [tokens, n_sum] expected")
+        if (y is None) != (a is None) or (z is None and entries is None) != (b is None) or (then is None) != (then_out is None) \
+                or (then_out is not None and tuple(then_out.shape) != (T, n)):
+            raise KernelError("parallel_sum: a result and its factor come together, and so do the norm and its output")
+        w2, e2, o2 = then if then is not None else (None, 0.0, 0.0)
+        vec = lambda t, what: self._f32_vec(t, n, what) if t is not None else None
+        rows = lambda t, what: (t.data_ptr(), _rows(t, what)) if t is not None else (None, 0)
+        self._call("hb_parallel_sum", x.data_ptr(), _rows(x, "residual"), *rows(y, "first result"), vec(a, "first factor"), *rows(z, "second result"),
+                   *rows(entries, "entries"), entry_weights.data_ptr() if entry_weights is not None else None, n_sum, vec(b, "second factor"),
+                   vec(vector, "vector"), vec(w2, "norm weight"), float(e2), float(o2), then_out.data_ptr() if then_out is not None else None,
+                   _code(then_out) if then_out is not None else 0, _rows(then_out, "norm output") if then_out is not None else 0, T, n, self._stream())
+        self.launches += 1
+
     def side_unit(self, s, tokens, table, col0: int, out, dim: int) -> None:
         """``out[t, :dim] = gelu_tanh(s[t, :dim]) * table[tokens[t], col0 : col0 + dim]``, zeros in ``out``'s further columns; ``s``
         float32, ``table`` row-major ``[vocab, columns]``."""
@@ -1373,12 +1410,20 @@ class Ops:
                    1 if append else 0, self.status.data_ptr(), self._stream())
         self.launches += 1
 
-    def latent_gather(self, cache, step, rank: int, rows, scratch_table) -> None:
-        """The latents of the step's sequences, from their first token on, page by page: ``rows`` bfloat16 ``[pages * 64, rank]``
+    @staticmethod
+    def latent_pages(step, window: Optional[int] = None) -> int:
+        """The pages of the step's sequences that its new tokens can see: all of them, or with a window those from the oldest
+        token on that a sequence's first new token sees."""
+        first = lambda n, new: max(0, n - new - int(window) + 1) // 64 if window else 0
+        return sum((n + 63) // 64 - first(n, new) for n, new in zip(step.host_len, step.host_new))
+
+    def latent_gather(self, cache, step, rank: int, rows, scratch_table, window: Optional[int] = None) -> None:
+        """The latents of the step's sequences, page by page, from their first token on or with a window from the first page
+        that counts (``latent_pages``): ``rows`` bfloat16 ``[pages * 64, rank]``
         (sequence b's pages follow those of the sequences in front of it; rows behind a sequence's end are zeros) and the page
-        table of that layout, ``scratch_table`` int32 ``[sequences, width]``."""
+        table of that layout, ``scratch_table`` int32 ``[sequences, width]`` (-1 for pages that do not count)."""
         self._dev(cache.v, rows, scratch_table)
-        pages = sum((n + 63) // 64 for n in step.host_len)
+        pages = self.latent_pages(step, window)
         if cache.v.dtype != torch.bfloat16 or rows.dtype != torch.bfloat16 or not rows.is_contiguous() or tuple(rows.shape) != (pages * 64, rank) \
                 or tuple(cache.v.shape[1:]) != (1, 64, rank) or not cache.v.is_contiguous():
             raise KernelError("latent_gather: bfloat16 cache [pages, 1, 64, rank] and rows [step pages * 64, rank] expected")
@@ -1386,24 +1431,24 @@ class Ops:
                 or scratch_table.shape[1] < (step.max_len + 63) // 64:
             raise KernelError("latent_gather: the scratch page table must be int32 [sequences, pages of the longest]")
         pt = step.page_tables[cache.group]
-        self._call("hb_latent_gather", cache.v.data_ptr(), pt.data_ptr(), pt.shape[1], step.seq_len.data_ptr(), step.num_seqs,
-                   (step.max_len + 63) // 64, rank, rows.data_ptr(), scratch_table.data_ptr(), scratch_table.shape[1], cache.v.shape[0],
+        self._call("hb_latent_gather", cache.v.data_ptr(), pt.data_ptr(), pt.shape[1], step.seq_len.data_ptr(), step.seq_pos0.data_ptr(),
+                   int(window or 0), step.num_seqs, (step.max_len + 63) // 64, rank, rows.data_ptr(), scratch_table.data_ptr(), scratch_table.shape[1], cache.v.shape[0],
                    self.status.data_ptr(), self._stream())
         self.launches += 1
 
-    def latent_scatter(self, kv, cache, step, heads: int, d: int, dr: int, dv: int, rank: int, k_out, v_out) -> None:
+    def latent_scatter(self, kv, cache, step, heads: int, d: int, dr: int, dv: int, rank: int, k_out, v_out, window: Optional[int] = None) -> None:
         """From ``kv`` bfloat16 ``[pages * 64, >= heads * (d + dv)]`` = ``[k_u (heads x d) | v (heads x dv)]`` per gathered row and the
         cached rotated key parts: ``k_out`` ``[pages, heads, 64, >= d + dr]`` = ``[k_u | k_r | zeros]`` and ``v_out`` ``[pages, heads, 64,
         >= dv]`` = ``[v | zeros]``, the paged layout of a cache with as many key/value heads as heads."""
         self._dev(kv, cache.k, k_out, v_out)
-        pages = sum((n + 63) // 64 for n in step.host_len)
+        pages = self.latent_pages(step, window)
         if any(t.dtype != torch.bfloat16 for t in (kv, cache.k, k_out, v_out)) or kv.shape[0] != pages * 64 or kv.stride(1) != 1 \
                 or not k_out.is_contiguous() or not v_out.is_contiguous() or tuple(k_out.shape[:3]) != (pages, heads, 64) \
                 or tuple(v_out.shape[:3]) != (pages, heads, 64) or tuple(cache.k.shape[1:]) != (1, 64, rank + dr):
             raise KernelError("latent_scatter: bfloat16 rows [step pages * 64, ..] and outputs [step pages, heads, 64, ..] expected")
         pt = step.page_tables[cache.group]
         self._call("hb_latent_scatter", kv.data_ptr(), _rows(kv, "keys and values"), cache.k.data_ptr(), pt.data_ptr(), pt.shape[1],
-                   step.seq_len.data_ptr(), step.num_seqs, (step.max_len + 63) // 64, heads, d, dr, dv, rank, k_out.shape[3], v_out.shape[3],
+                   step.seq_len.data_ptr(), step.seq_pos0.data_ptr(), int(window or 0), step.num_seqs, (step.max_len + 63) // 64, heads, d, dr, dv, rank, k_out.shape[3], v_out.shape[3],
                    k_out.data_ptr(), v_out.data_ptr(), cache.k.shape[0], self._stream())
         self.launches += 1
 
@@ -1561,18 +1606,19 @@ class Ops:
 
     SCORINGS = {"softmax_chosen": 0, "sigmoid": 1}
 
-    def moe_route(self, h, w_router, top: int, experts, weights, scoring: str = "softmax_chosen") -> None:
+    def moe_route(self, h, w_router, top: int, experts, weights, scoring: str = "softmax_chosen", bias=None) -> None:
         """Per token the ``top`` experts with the largest router logits (``w_router`` float32 ``[experts, width]``, logits in
         32-bit) into ``experts`` int32 ``[tokens, top]`` and the softmax over those logits into ``weights`` float32; ``scoring``
-        "sigmoid": the chosen logits' sigmoids instead, not divided by their sum."""
-        self._dev(h, w_router, experts, weights)
+        "sigmoid": the chosen logits' sigmoids instead, not divided by their sum.  ``bias`` float32 ``[experts]`` is part of the logits."""
+        self._dev(h, w_router, experts, weights, bias)
         T, W = h.shape
         E = w_router.shape[0]
         if w_router.dtype != torch.float32 or not w_router.is_contiguous() or w_router.shape[1] != W or experts.dtype != torch.int32 \
                 or weights.dtype != torch.float32 or tuple(experts.shape) != (T, top) or tuple(weights.shape) != (T, top) \
                 or not experts.is_contiguous() or not weights.is_contiguous():
             raise KernelError("moe_route: float32 router [experts, width], int32 and float32 [tokens, top] outputs expected")
-        self._call("hb_moe_route", h.data_ptr(), _code(h), _rows(h, "router input"), w_router.data_ptr(), experts.data_ptr(),
+        self._call("hb_moe_route", h.data_ptr(), _code(h), _rows(h, "router input"), w_router.data_ptr(),
+                   self._f32_vec(bias, E, "router bias") if bias is not None else None, experts.data_ptr(),
                    weights.data_ptr(), T, W, E, int(top), self.SCORINGS[scoring], self._stream())
         self.launches += 1
 
@@ -1589,10 +1635,10 @@ class Ops:
         numbers from the stack's size on are identity experts, whose result is ``h[t]`` itself.  ``unit`` "silu_glu": ``silu(gate) * up``
         between the products.  ``weigh`` "input": an expert is fed ``weights[t, k] * h[t]`` and its result is added as it is.
         ``out`` None: no sum; returns the experts' results, float32 ``[tokens * top, width]`` (engine scratch), for a caller whose
-        own kernel adds a token's rows (``weigh`` "input" only)."""
+        own kernel adds a token's rows (with their weights unless ``weigh`` is "input")."""
         self._dev(h, experts, weights, w_gate, w_up, w_down, out)
-        if (out is None and (weigh != "input" or identity)) or weigh not in ("input", "output") or (weigh == "input" and identity):
-            raise KernelError("moe_experts: results are handed on unsummed only when the weights went into the inputs; identity experts weigh outputs")
+        if (out is None and identity) or weigh not in ("input", "output") or (weigh == "input" and identity):
+            raise KernelError("moe_experts: identity experts have their results weighted and summed here")
         T, W = h.shape
         E, F = w_gate.shape[0], w_gate.shape[1]
         top = experts.shape[1]

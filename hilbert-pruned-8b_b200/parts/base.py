@@ -24,6 +24,8 @@ What a part must provide:
   head dimensions by position-dependent angles (the kernels then turn queries and keys
   themselves), else ``apply(q, k, step)`` which turns them in place; see ``PositionEncoding``.
 * residual gates: ``logits(h, step)`` (32-bit, without the bias) and ``bias``.
+* residual scales: ``factors`` (32-bit ``[width]``), one factor per channel of a sublayer's result.
+* stream vectors: ``vector(i)`` (32-bit ``[width]``), what a plan entry adds to every token's stream in front of itself.
 * token sides: ``forward(h, x, step, copy=None)``, adding to the 32-bit stream ``x``.
 * blocks (``parts/block.py``): ``ROLES``, ``named_parts()``, ``cache_need()``, ``state_need()``,
   ``forward(x, step, cache, state, append)``.
@@ -170,6 +172,11 @@ class FeedForward(Part):
 
     sums_entries = False
 
+    # ``weighs_entries = True`` (may depend on the part's options): ``forward_weighted(h, step)`` returns ``(rows, n, weights, base)``: the
+    # result of token t is ``base[t] + sum_k weights[t, k] * rows[t * n + k]``, all 32-bit, ``base`` None: nothing, for a caller whose own
+    # kernel forms that sum.
+    weighs_entries = False
+
     folds_norms = False
     can_overwrite = False
 
@@ -290,4 +297,6 @@ BLOCKS = Registry("block")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
 RESIDUAL_GATES = Registry("residual gate")
+RESIDUAL_SCALES = Registry("residual scale")
+STREAM_VECTORS = Registry("stream vectors")
 TOKEN_SIDES = Registry("token side input")

@@ -14,7 +14,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, RESIDUAL_GATES, TOKEN_FILTERS, TOKEN_SIDES, CacheNeed, Registry,
+from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, RESIDUAL_GATES, RESIDUAL_SCALES, TOKEN_FILTERS, TOKEN_SIDES, CacheNeed, Registry,
                    StateNeed)
 
 
@@ -54,6 +54,10 @@ class Block:
     # prepared, the block runs its first norm), ``prepare_next`` what the next block's
     # ``fold_request`` said (None: nobody asks).  Other blocks are called without them.
     folds_norms = False
+
+    # A block with ``adds_vector = True`` (one with ``folds_norms``) also takes ``vector=``: 32-bit ``[width]``, added to every token's
+    # stream behind the block's own sum and before what ``prepare_next`` asks for is made of it (``PlanEntry.adds``).
+    adds_vector = False
 
     def fold_request(self, step):
         """What the block in front has to prepare so that this block need not run its first
@@ -421,3 +425,64 @@ class PostNormSumBlock(Block):
         if self.side is not None:
             self.side.forward(h, x, step, copy=ahead)
         return COPIED if ahead is not None else None
+
+
+@BLOCKS.register("parallel_prenorm")
+class ParallelPreNormBlock(Block):
+    """Both sublayers side by side behind one norm: ``h = norm(x)``, ``x += s_a * mixer(h) + s_b * feed_forward(h)`` with a factor per
+    channel on each result (a layer without a feed-forward: the first term alone).  The mixer and the feed-forward leave their
+    results in 32-bit buffers of their own; a mixture of experts hands its experts' results on unsummed
+    (``FeedForward.weighs_entries``).  One kernel forms the whole sum, adds the vector that the next plan entry adds in front of
+    itself (``adds_vector``) and makes the next layer's norm output from the new row, where that layer asks for it
+    (``fold_request`` / ``prepare_next``, the protocol of the sandwich block)."""
+
+    ROLES = {"norm": NORMS, "mixer": MIXERS, "mixer_scale": RESIDUAL_SCALES, "feed_forward": FEED_FORWARDS, "feed_forward_scale": RESIDUAL_SCALES}
+    OPTIONAL = ("feed_forward", "feed_forward_scale")
+    folds_norms = True
+
+    def __init__(self, layer_spec, ctx):
+        super().__init__(layer_spec, ctx)
+        p = self.parts
+        self.norm, self.mixer, self.mixer_scale = p["norm"], p["mixer"], p["mixer_scale"]
+        self.ff, self.ff_scale = p.get("feed_forward"), p.get("feed_forward_scale")
+        if (self.ff is None) != (self.ff_scale is None):
+            raise ValueError(f"layer {layer_spec.prefix!r}: a feed-forward and the factors on its result come together")
+        self.fuse_norms = True              # tests switch these two off to run every norm as a kernel of its own,
+        self.fuse_entries = True            # and to let a mixture of experts sum its results itself
+
+    @property
+    def adds_vector(self) -> bool:
+        return self.fuse_norms
+
+    def _h(self, step, size: int):
+        return self.ctx.workspace.buffer("block.h", (self.ctx.max_step_tokens, size), self.ctx.dtype)[:step.num_tokens]
+
+    def fold_request(self, step):
+        size = getattr(self.norm, "size", None)
+        if not self.fuse_norms or size is None:
+            return None
+        request = self.norm.fold_request(self._h(step, size))
+        return NormAhead(request) if request is not None else None
+
+    def forward(self, x, step, cache, state, append: bool, prepared=None, prepare_next=None, vector=None):
+        ws, cap, T = self.ctx.workspace, self.ctx.max_step_tokens, step.num_tokens
+        h = self._h(step, x.shape[1])
+        if prepared is not NORMED:
+            self.norm.forward(x, h)
+        y = ws.buffer("block.branch", (cap, x.shape[1]), torch.float32)[:T]
+        SandwichBlock._run(self.mixer, y, (h, y, step, cache, state, append))
+        terms = {}
+        if self.ff is not None:
+            if self.fuse_entries and getattr(self.ff, "weighs_entries", False):
+                rows, n, weights, base = self.ff.forward_weighted(h, step)
+                terms = {"entries": rows, "n_sum": n, "entry_weights": weights, "z": base}
+            else:
+                z = ws.buffer("block.second_branch", (cap, x.shape[1]), torch.float32)[:T]
+                SandwichBlock._run(self.ff, z, (h, z, step))
+                terms = {"z": z}
+            terms["b"] = self.ff_scale.factors
+        ahead = prepare_next if (self.fuse_norms and isinstance(prepare_next, NormAhead) and tuple(prepare_next[3].shape) == tuple(x.shape)) else None
+        if ahead is not None:
+            terms.update(then=(ahead[0], ahead[2], ahead[1]), then_out=ahead[3])
+        self.ctx.ops.parallel_sum(x, y=y, a=self.mixer_scale.factors, vector=vector, **terms)
+        return NORMED if ahead is not None else None

@@ -9,7 +9,9 @@ h's unrotated key is ``Wuk_h c`` and its value ``Wuv_h c``; its score for a key 
 
 Options beside that form: ``q_rank``: the queries come through a latent of their own, ``q = Wuq rmsnorm(Wdq h)`` (tensors ``dq``,
 ``dq.norm``, ``uq`` in the place of ``q``); ``shares_cache``: the layer has no ``Wdkv`` and reads the latents and key parts that an
-earlier layer of the same rank and rotation cached (its plan entry's ``cache_of``), with its own ``Wuk`` and ``Wuv``.
+earlier layer of the same rank and rotation cached (its plan entry's ``cache_of``), with its own ``Wuk`` and ``Wuv``; ``window`` n: a
+query sees the n newest tokens only, itself included; ``sink``: a learned number per head (tensor ``sink``) whose exponential is one
+more term of the softmax's sum, with no key and no value.
 
 Only ``c`` and the rotated key part are cached.  The up projections are folded around the attention
 instead of being applied to the cache: with ``q'_h = [Wuk_h^T q_u | q_r]`` the score is ``q'_h . [c | k_r]``
@@ -19,7 +21,7 @@ the library's softmax attention over a paged cache group (``softmax_attention``)
 
 That folded form is what a step of few tokens runs (decoding: the cache is read once, for all heads).  A bfloat16
 step that brings many tokens writes the keys and values of every head out instead, for its sequences from their
-first token on, into a scratch cache of the ordinary paged layout with as many key/value heads as heads: key
+first token on (with a window: from the page of the oldest token that the step's first new token sees), into a scratch cache of the ordinary paged layout with as many key/value heads as heads: key
 ``[Wuk_h c | k_r]`` of ``d + dr`` numbers, value ``Wuv_h c``, each padded with zeros to a head size the tensor-core
 prompt kernel is built for (``written_out``).  The products of the attention are then several times smaller than
 with ``rank + dr`` numbers per key, and the two per-head products become one ordinary matrix product.
@@ -51,6 +53,9 @@ class LatentAttention(Mixer):
         self.scale = float(p["scale"])
         self.eps = float(p["eps"])
         self.head_gate = bool(p.get("head_gate", False))
+        self.window = int(p["window"]) if p.get("window") is not None else None
+        self.sink = bool(p.get("sink", False))
+        self.sink_logits = None
         pos = p.get("position")
         self.position = ctx.shared_part(POSITION_ENCODINGS, pos) if pos is not None else None
         self.graph_safe = getattr(self.position, "graph_safe", True)
@@ -81,6 +86,8 @@ class LatentAttention(Mixer):
         out += [ParamSpec("uk", (H * self.d, self.rank)), ParamSpec("uv", (H * self.dv, self.rank)), ParamSpec("o", (W, H * self.dv))]
         if self.head_gate:
             out.append(ParamSpec("g", (H, W)))
+        if self.sink:
+            out.append(ParamSpec("sink", (H,), kind="vector", init="zeros"))
         return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -95,6 +102,8 @@ class LatentAttention(Mixer):
             self.w_uq = pack(t["uq"].contiguous())
             self.q_weight = t["dq.norm"].reshape(-1).to(torch.float32).contiguous()
         self.w_o = pack(t["o"].contiguous())
+        if self.sink:
+            self.sink_logits = t["sink"].reshape(-1).to(torch.float32).contiguous()
         # per head [inputs, outputs]: the key up-projection is stored that way already (it is applied transposed, to the query)
         self.w_uk = t["uk"].reshape(H, self.d, self.rank).contiguous()
         self.w_uv = t["uv"].reshape(H, self.dv, self.rank).transpose(1, 2).contiguous()
@@ -113,7 +122,7 @@ class LatentAttention(Mixer):
         return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_uq, self.w_uk, self.w_uv, self.w_o) if w is not None)
 
     def cache_need(self) -> CacheNeed:
-        return CacheNeed(1, self.key_dim, None, v_head_dim=self.rank)
+        return CacheNeed(1, self.key_dim, self.window, v_head_dim=self.rank)
 
     def forward(self, h, residual, step, cache, state, append: bool, accumulate: bool = True):
         if append and self.shares_cache:
@@ -145,7 +154,7 @@ class LatentAttention(Mixer):
         ops.latent_prepare(q_raw, down, H, d, dr, rank, self.c_weight, self.eps, table, rot, q, cache, step, append)
         ops.head_linear(q_raw, d + dr, self.w_uk, q, self.key_dim, d, rank)
         mixed = ws.buffer("latent_attention.mixed", (cap, H * rank), torch.float32)[:T]
-        softmax_attention(self.ctx, q, H, 1, self.key_dim, rank, cache, step, self.scale, None, 0, mixed)
+        softmax_attention(self.ctx, q, H, 1, self.key_dim, rank, cache, step, self.scale, self.window, 0, mixed, sink=self.sink_logits)
         attn = ws.buffer("latent_attention.out", (cap, H * dv), self.ctx.dtype)[:T]
         ops.head_linear(mixed, rank, self.w_uv, attn, dv, rank, dv, gate=gate)
         ops.linear(attn, self.w_o, residual, accumulate=accumulate)
@@ -160,20 +169,20 @@ class LatentAttention(Mixer):
         H, d, dr, dv, rank, D, DV = self.heads, self.d, self.dr, self.dv, self.rank, self.flat_d, self.flat_dv
         q = ws.buffer("latent_attention.q_flat", (cap, H * D), torch.bfloat16)[:T]
         ops.latent_prepare(q_raw, down, H, d, dr, rank, self.c_weight, self.eps, table, rot, q, cache, step, append, whole_heads=D)
-        pages = sum((n + 63) // 64 for n in step.host_len)
+        pages = ops.latent_pages(step, self.window)
         width = (step.max_len + 63) // 64
         rows = ws.buffer("latent_attention.flat_c", (pages * 64, rank), torch.bfloat16)
         scratch_table = ws.buffer("latent_attention.flat_pages", (step.num_seqs, width), torch.int32)
-        ops.latent_gather(cache, step, rank, rows, scratch_table)
+        ops.latent_gather(cache, step, rank, rows, scratch_table, window=self.window)
         kv = ws.buffer("latent_attention.flat_kv", (pages * 64, H * (d + dv)), torch.bfloat16)
         ops.linear(rows, self.w_ukv, kv)
         flat = _WrittenOut(ws.buffer("latent_attention.flat_k", (pages, H, 64, D), torch.bfloat16),
                            ws.buffer("latent_attention.flat_v", (pages, H, 64, DV), torch.bfloat16), len(step.page_tables))
-        ops.latent_scatter(kv, cache, step, H, d, dr, dv, rank, flat.k, flat.v)
+        ops.latent_scatter(kv, cache, step, H, d, dr, dv, rank, flat.k, flat.v, window=self.window)
         step.page_tables.append(scratch_table)              # the scratch cache is one more group of this step
         try:
             attn = ws.buffer("latent_attention.out_flat", (cap, H * DV), torch.bfloat16)[:T]
-            softmax_attention(self.ctx, q, H, H, D, DV, flat, step, self.scale, None, 0, attn, gate=gate)
+            softmax_attention(self.ctx, q, H, H, D, DV, flat, step, self.scale, self.window, 0, attn, gate=gate, sink=self.sink_logits)
         finally:
             step.page_tables.pop()
         ops.linear(attn, self.w_o_flat, residual, accumulate=accumulate)

@@ -16,7 +16,8 @@ identity experts, which hand the token's input back (times the weight) and have 
 by ``sigmoid(W_sg h)``, one number per token (tensor ``shared.sg`` ``[1, width]``).  ``router`` "sigmoid": the ``top`` largest
 logits as in the plain form, weighted by their sigmoids, not divided by anything.  ``unit`` "silu_glu": an expert is
 ``W_down (silu(W_gate h) * (W_up h))``.  ``weigh`` "input": an expert is fed ``weight * h`` and its result is added as it is
-(evaluated as ``W (w h) = w (W h)`` in front of the activation, in 32-bit).
+(evaluated as ``W (w h) = w (W h)`` in front of the activation, in 32-bit).  ``router_bias``: the router's logits have a bias (tensor
+``router.b``), which counts for the choice and for the weights; for the routers "top_logits" and "sigmoid".
 
 Tensors below the part's prefix: ``router``, ``e<i>.gate|up|down``, ``shared.gate|up|down``.  The
 experts' matrices are stacked at load time; the routed products gather their rows on the device
@@ -65,11 +66,17 @@ class MixtureOfExperts(FeedForward):
             raise ValueError(f"moe: top {self.top} of {self.n_outputs} experts")
         if self.weigh == "input" and self.identity:
             raise ValueError("moe: identity experts have their results weighted")
-        if self.unit == "silu_glu" and self.shared_ff:
-            raise ValueError("moe: no shared expert is built for the unit 'silu_glu'")
+        self.router_bias = bool(p.get("router_bias", False))
+        if self.router_bias and self.router == "scores":
+            raise ValueError("moe: the router 'scores' has a correction, not a bias")
+        if self.unit == "silu_glu" and self.shared_gate:
+            raise ValueError("moe: the gate on the shared expert belongs to the unit 'gelu'")
         self.glu = self.unit != "gelu"                        # two matrices in front of the activation
         # the experts' results can be handed on unsummed (one row per token and chosen expert)
         self.sums_entries = self.weigh == "input" and not self.shared_ff
+        # or with their weights and the shared expert's result beside them
+        self.weighs_entries = not self.identity
+        self.b_router = None
         self.correction = None
         self.gate_col = None
         self.w_router = self.w_gate = self.w_up = self.w_down = self.ws_gate_up = self.ws_down = None
@@ -78,6 +85,8 @@ class MixtureOfExperts(FeedForward):
         W, F = self.hidden, self.ff
         glu = self.glu
         out = [ParamSpec("router", (self.n_outputs, W))]
+        if self.router_bias:
+            out.append(ParamSpec("router.b", (self.n_outputs,), kind="vector", init="zeros"))
         if self.router == "scores":
             out.append(ParamSpec("correction", (self.n_outputs,), kind="vector", init="zeros"))
         for e in range(self.n_experts):
@@ -92,6 +101,8 @@ class MixtureOfExperts(FeedForward):
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         t, E = tensors, self.n_experts
         self.w_router = t["router"].to(torch.float32).contiguous()
+        if self.router_bias:
+            self.b_router = t["router.b"].reshape(-1).to(torch.float32).contiguous()
         glu = self.glu
         self.w_gate = torch.stack([t[f"e{e}.gate"] for e in range(E)]).contiguous() if glu else None
         self.w_up = torch.stack([t[f"e{e}.up"] for e in range(E)]).contiguous()
@@ -108,7 +119,8 @@ class MixtureOfExperts(FeedForward):
                 pad = (-(self.gate_col + 1)) % 8
                 if pad:
                     rows.append(torch.zeros(pad, self.hidden, dtype=rows[0].dtype, device=rows[0].device))
-            self.ws_gate_up = pack(torch.cat(rows, dim=0).contiguous())
+            # (the plain gated unit is the epilogue of its first product: linear_swiglu)
+            self.ws_gate_up = pack(torch.cat(rows, dim=0).contiguous(), swiglu=self.unit == "silu_glu")
             self.ws_down = pack(t["shared.down"].contiguous())
 
     def weight_bytes(self) -> int:
@@ -119,7 +131,15 @@ class MixtureOfExperts(FeedForward):
 
     def forward_entries(self, h, step):
         """``(rows, top)``: the chosen experts' results, 32-bit ``[tokens * top, width]``, whose sum per token is the result."""
-        return self._experts(h, step, None, False), self.top
+        return self._experts(h, step, None, False)[0], self.top
+
+    def forward_weighted(self, h, step):
+        rows, weights = self._experts(h, step, None, False)
+        base = None
+        if self.shared_ff:
+            base = self.ctx.workspace.buffer("moe.shared_out", (self.ctx.max_step_tokens, self.hidden), torch.float32)[: step.num_tokens]
+            self._shared(h, base, step, accumulate=False)
+        return rows, self.top, weights if self.weigh == "output" else None, base
 
     def _experts(self, h, step, residual, accumulate: bool):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
@@ -128,25 +148,36 @@ class MixtureOfExperts(FeedForward):
         if self.router == "scores":
             ops.moe_route_scores(h, self.w_router, self.correction, self.top, self.groups, self.keep, experts, weights)
         else:
-            ops.moe_route(h, self.w_router, self.top, experts, weights, scoring="sigmoid" if self.router == "sigmoid" else "softmax_chosen")
+            ops.moe_route(h, self.w_router, self.top, experts, weights, scoring="sigmoid" if self.router == "sigmoid" else "softmax_chosen",
+                          bias=self.b_router)
         if self.unit == "gelu":
-            return ops.moe_experts(h, experts, weights, self.w_up, None, self.w_down, 0.0, 0.0, residual, accumulate, ws, cap,
+            rows = ops.moe_experts(h, experts, weights, self.w_up, None, self.w_down, 0.0, 0.0, residual, accumulate, ws, cap,
                                    tag=".gelu", identity=self.identity > 0, weigh=self.weigh)
-        return ops.moe_experts(h, experts, weights, self.w_gate, self.w_up, self.w_down, self.limit, self.alpha, residual, accumulate, ws, cap,
-                               unit=self.unit, weigh=self.weigh)
+        else:
+            rows = ops.moe_experts(h, experts, weights, self.w_gate, self.w_up, self.w_down, self.limit, self.alpha, residual, accumulate, ws, cap,
+                                   unit=self.unit, weigh=self.weigh)
+        return rows, weights
 
     def forward(self, h, residual, step, accumulate: bool = True):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         self._experts(h, step, residual, accumulate)
         if self.shared_ff:
-            S = self.shared_ff
+            self._shared(h, residual, step, accumulate=True)
+
+    def _shared(self, h, out, step, accumulate: bool) -> None:
+        """The shared expert's result, added to ``out`` or written there."""
+        ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
+        S = self.shared_ff
+        act = ws.buffer("moe.shared_act", (cap, S), self.ctx.dtype)[:T]
+        if self.unit == "silu_glu":
+            ops.linear_swiglu(h, self.ws_gate_up, act, ws, cap)
+        else:
             first = self.ws_gate_up.shape[0]
             gu = ws.buffer(f"moe.shared_first.{first}", (cap, first), torch.float32)[:T]
             ops.linear(h, self.ws_gate_up, gu)
-            act = ws.buffer("moe.shared_act", (cap, S), self.ctx.dtype)[:T]
             if self.unit == "gelu":
                 # sigmoid(W_sg h) * (W_down act) = W_down (sigmoid(W_sg h) * act): the gate multiplies the rows the product reads
                 ops.gelu_unit(gu, act, "erf", row_gate=self.gate_col)
             else:
                 ops.glu_clamp(gu[:, : 2 * S], act, self.shared_limit, self.alpha)
-            ops.linear(act, self.ws_down, residual, accumulate=True)
+        ops.linear(act, self.ws_down, out, accumulate=accumulate)

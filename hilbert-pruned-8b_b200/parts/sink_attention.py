@@ -4,7 +4,7 @@ root mean square after the rotation (or, ``qk_norm_weight``, divided by it and m
 of the head's size, shared by the heads, BEFORE the rotation), key and value heads of different sizes,
 softmax weights mixed between the heads, values mixed with those of an earlier layer, and
 (``head_gate``) each head's result multiplied by ``sigmoid(Wg h)_head``, one number per token and head,
-before the output projection.  ``out_bias`` (default: as ``bias``) says whether the output projection has
+before the output projection, or (``element_gate``) every element of the results by its own ``sigmoid(Wg h)``.  ``out_bias`` (default: as ``bias``) says whether the output projection has
 a bias too.  ``chunk`` (instead of a window): positions are cut into runs of ``chunk`` from the sequence's start and a query
 sees only the keys of its own run.  ``sink``: a learned number per head (tensor ``sink``) whose exponential is one more
 term of the softmax's sum, with no key and no value.  ``v_from_k``: no value projection; the values are the keys as
@@ -60,6 +60,9 @@ class SinkAttention(Mixer):
         if self.qk_unit_norm and self.qk_norm_weight:
             raise ValueError("attention: queries and keys get one norm, behind the rotation or in front of it")
         self.head_gate = bool(p.get("head_gate", False))
+        self.element_gate = bool(p.get("element_gate", False))
+        if self.head_gate and self.element_gate:
+            raise ValueError("attention: one gate, per head or per element")
         self.out_bias = bool(p.get("out_bias", p.get("bias", False)))
         self.eps = float(p.get("eps", 1e-6))
         self.talk = bool(p.get("talk", False))
@@ -76,7 +79,8 @@ class SinkAttention(Mixer):
         self.graph_safe = getattr(self.position, "graph_safe", True)
         self.q_width, self.k_width, self.v_width = self.heads * self.head_dim, self.kv_heads * self.head_dim, self.kv_heads * self.v_dim
         self.gate_at = self.q_width + self.k_width + (0 if self.v_from_k else self.v_width)
-        self.proj_width = self.gate_at + (self.heads if self.head_gate else 0)
+        self.gate_width = self.heads if self.head_gate else self.heads * self.v_dim if self.element_gate else 0
+        self.proj_width = self.gate_at + self.gate_width
         self.proj_ld = (self.proj_width + 7) // 8 * 8
         self.out_width = self.heads * self.v_dim
         self.w_qkv = self.w_o = self.b_qkv = self.talk_matrix = self.v_lambda = self.norm_weights = self.sink_logits = None
@@ -96,8 +100,8 @@ class SinkAttention(Mixer):
             out.append(ParamSpec("o.b", (W,), kind="vector", init="zeros"))
         if self.qk_norm_weight:
             out += [ParamSpec("q.norm", (self.head_dim,), kind="vector", init="ones"), ParamSpec("k.norm", (self.head_dim,), kind="vector", init="ones")]
-        if self.head_gate:
-            out.append(ParamSpec("g", (self.heads, W)))
+        if self.gate_width:
+            out.append(ParamSpec("g", (self.gate_width, W)))
         if self.talk:
             out.append(ParamSpec("talk", (self.heads, self.heads)))
         if self.v_mix is not None:
@@ -111,7 +115,7 @@ class SinkAttention(Mixer):
         v = None if self.v_from_k else t["v"]
         if q.dtype != k.dtype or (v is not None and v.dtype != q.dtype):
             raise ValueError("attention: q, k and v projections are stored in different dtypes")
-        rows = [q, k] + ([] if v is None else [v]) + ([t["g"]] if self.head_gate else [])
+        rows = [q, k] + ([] if v is None else [v]) + ([t["g"]] if self.gate_width else [])
         if len({r.dtype for r in rows}) != 1:
             raise ValueError("attention: the input projections are stored in different dtypes")
         if self.proj_ld > self.proj_width:
@@ -170,7 +174,7 @@ class SinkAttention(Mixer):
         ops.qkv_prepare(proj, self.b_qkv, table, rot, H, G, d, dv, self.qk_unit_norm, self.eps, q, cache, step, append,
                         self.v_lambda, v_first, v_mode, norm_weights=self.norm_weights, interleaved=self.interleaved, v_from_k=self.v_from_k)
         ones = _BIAS_PAD if self.out_bias else 0
-        gate = proj[:, self.gate_at: self.gate_at + H] if self.head_gate else None
+        gate = proj[:, self.gate_at: self.gate_at + self.gate_width] if self.gate_width else None
         attn = ws.buffer("sink_attention.out", (cap, self.out_width + ones), self.ctx.dtype)[:T]
         softmax_attention(self.ctx, q, H, G, d, dv, cache, step, self.scale, self.window, self.keep_first, attn, ones=ones, gate=gate,
                           talk_matrix=self.talk_matrix if self.talk else None, use_heads_kernel=self.use_heads_kernel,
@@ -183,7 +187,7 @@ def softmax_attention(ctx, q, H: int, G: int, d: int, dv: int, cache, step, scal
     """Softmax attention of the step's queries ``q [tokens, H * d]`` over the cached keys and values of ``cache`` (``G``
     key/value heads of sizes ``d`` and ``dv``), by whichever kernel takes the step: ``out [tokens, H * dv + ones]`` (the
     dtype of the products, or 32-bit) receives the normalised results, mixed between the heads by ``talk_matrix``, each
-    head's times ``sigmoid(gate[t, head])``, and ``ones`` more columns (a one, then zeros).  ``chunk`` (instead of a window) and
+    head's times ``sigmoid(gate[t, head])`` (``gate`` ``[tokens, H * dv]``: every element's times its own), and ``ones`` more columns (a one, then zeros).  ``chunk`` (instead of a window) and
     ``sink`` (float32 ``[H]``) as the kernels take them.  Any part that has put its keys
     and values into a paged cache group can call it."""
     ops, ws, T, cap = ctx.ops, ctx.workspace, step.num_tokens, ctx.max_step_tokens

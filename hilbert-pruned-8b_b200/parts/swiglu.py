@@ -86,11 +86,29 @@ class GatedGelu(FeedForward):
     def weight_bytes(self) -> int:
         return sum(w.numel() * w.element_size() for w in (self.w_gate_up, self.w_down))
 
+    def _unit(self, gate_up, act) -> None:
+        self.ctx.ops.gelu_unit(gate_up, act, "tanh_gated")
+
     def forward(self, h, residual, step, accumulate: bool = True):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         first = self.w_gate_up.shape[0]
         gu = ws.buffer(f"gated_gelu.gate_up.{first}", (cap, first), torch.float32)[:T]
         ops.linear(h, self.w_gate_up, gu)
         act = ws.buffer("gated_gelu.act", (cap, self.inter), self.ctx.dtype)[:T]
-        ops.gelu_unit(gu, act, "tanh_gated")
+        self._unit(gu, act)
         ops.linear(act, self.w_down, residual, accumulate=accumulate)
+
+
+@FEED_FORWARDS.register("clamped_glu")
+class ClampedGLU(GatedGelu):
+    """``residual += Wd (g sigmoid(alpha g) (u + 1))`` with ``g = min(Wg h, limit)`` and ``u = clamp(Wu h, -limit, limit)``; ``alpha`` is 1.702
+    unless the spec says otherwise.  Gate and up weights are one matrix product with a 32-bit result; the activation reads it
+    unrounded."""
+
+    def __init__(self, spec, ctx):
+        super().__init__(spec, ctx)
+        self.limit = float(spec.params["limit"])
+        self.alpha = float(spec.get("alpha", 1.702))
+
+    def _unit(self, gate_up, act) -> None:
+        self.ctx.ops.glu_clamp(gate_up[:, : 2 * self.inter], act, self.limit, self.alpha)
