@@ -7,6 +7,7 @@
     python bench.py --design vuladra      # a line of its own: the Vuladra design beside Pogezen layers of equal size
     python bench.py --design tonovik      # a line of its own: the Tonovik design beside Vuladra layers of equal size
     python bench.py --design moponex      # a line of its own: the Moponex design beside Vuladra layers of equal size
+    python bench.py --design mirorax      # a line of its own: the Mirorax design beside Tonovik and Moponex layers of equal size
     python bench.py --design ridotar      # a line of its own: the Ridotar design beside Tonovik and Moponex layers of equal size
 
 Prints ONE JSON line.  A step is one decode step of a batch of 8 sequences whose caches hold
@@ -516,6 +517,24 @@ def ridotar_config(z):
                        {"type": "latent_attention", "mixer": dict(lat, kv_from=2), "mlp": moe}]}
 
 
+# --design mirorax: four Mirorax layers (attention over cached latents with a window and a sink + clamped dense unit; causal
+# attention without positions, gated per element + mixture of experts; the latents + mixture of experts; the causal attention +
+# dense; the middle two form a run of layers with one pass) beside four Tonovik layers (the like of the latents, of a softmax
+# attention with gates and of a dense feed-forward) and four Moponex layers (the like of the mixture of experts with a shared
+# expert, and of an attention with a sink), at the same width, heads, head size and window.  The latents have Tonovik's ranks;
+# the experts are Moponex's 16 of a quarter of the dense feed-forward's size, two chosen, with a shared expert of that size.
+def mirorax_config(z):
+    W, hd = z["width"], z["head_dim"]
+    lat = {"type": "latent_attention", "mixer": {
+        "heads": z["heads"], "dim": hd, "rot_dim": hd // 2, "vdim": hd, "kv_rank": 4 * hd, "scale": (1.5 * hd) ** -0.5,
+        "mask": {"size": DESIGN_WINDOW}, "rot": {"base": 10000.0, "dims": hd // 2}}}
+    att = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": hd, "vdim": hd, "scale": hd ** -0.5}}
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "router": {"experts": VULADRA_EXPERTS, "top": VULADRA_TOP}, "expert": {"ff": z["ff"] // 4}, "shared": {"ff": z["ff"] // 4}}
+    return {"architecture": "Mirorax", "norm": {"eps": 1e-6}, "loop": {"start": 1, "stop": 3, "times": 1}, "vocab": DESIGN_VOCAB, "width": W,
+            "layers": [dict(lat, mlp=dense), dict(att, mlp=moe), dict(lat, mlp=moe), dict(att, mlp=dense)]}
+
+
 def llama_like_config(z):
     return dict(MODEL_8B, hidden_size=z["width"], num_hidden_layers=4, intermediate_size=z["ff"], vocab_size=DESIGN_VOCAB,
                 num_attention_heads=z["heads"], num_key_value_heads=z["kv"], head_dim=z["head_dim"], tie_word_embeddings=True)
@@ -564,7 +583,10 @@ def design_comparison(a) -> int:
     out = {}
     for size, z in DESIGN_SIZES.items():
         row = {}
-        if a.design == "ridotar":
+        if a.design == "mirorax":
+            pair = (("mirorax", hb.MiroraxConfig.from_dict(mirorax_config(z))), ("tonovik", hb.TonovikConfig.from_dict(tonovik_config(z))),
+                    ("moponex", hb.MoponexConfig.from_dict(moponex_config(z))))
+        elif a.design == "ridotar":
             pair = (("ridotar", hb.RidotarConfig.from_dict(ridotar_config(z))), ("tonovik", hb.TonovikConfig.from_dict(tonovik_config(z))),
                     ("moponex", hb.MoponexConfig.from_dict(moponex_config(z))))
         elif a.design == "moponex":
@@ -606,7 +628,7 @@ def design_comparison(a) -> int:
             del llm, eng, seqs
             torch.cuda.empty_cache()
         out[size] = row
-    names = {"ridotar": "Ridotar layers beside Tonovik and Moponex layers", "moponex": "Moponex layers beside Vuladra layers", "tonovik": "Tonovik layers beside Vuladra layers", "vuladra": "Vuladra layers beside Pogezen layers",
+    names = {"mirorax": "Mirorax layers beside Tonovik and Moponex layers", "ridotar": "Ridotar layers beside Tonovik and Moponex layers", "moponex": "Moponex layers beside Vuladra layers", "tonovik": "Tonovik layers beside Vuladra layers", "vuladra": "Vuladra layers beside Pogezen layers",
              "pogezen": "Pogezen layers beside Llama layers"}[a.design]
     print(json.dumps({"metric": f"{names} of equal size: prefill of one 2048-token prompt and decode "
                                 f"steps of batch {batch} at context {context}, four layers, random weights",
@@ -711,7 +733,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--workload", choices=("8b", "3b", "1b"), default="8b",
                     help="8b: the default line; 3b, 1b: the generation workloads at those shapes (--steps = repeats)")
-    ap.add_argument("--design", choices=("pogezen", "vuladra", "tonovik", "moponex", "ridotar"), default=None,
+    ap.add_argument("--design", choices=("pogezen", "vuladra", "tonovik", "moponex", "ridotar", "mirorax"), default=None,
                     help="a line of its own: this design's layers beside layers of equal size of the closest other designs (prefill, decode, "
                          "device time per kernel); the default workload is not run")
     ap.add_argument("--timeline", action="store_true",

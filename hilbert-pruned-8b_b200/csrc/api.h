@@ -130,6 +130,20 @@ int hb_head_mix_splits(const float* partial, const float* ml, const float* mix, 
                        int n_heads, int n_kv_heads, int v_dim, int splits, int ones, const float* gate, long long ldg, int gate_per, void* stream);
 // Flash-style on the tensor cores for steps of many tokens (bfloat16, head sizes 64 or 128); out float32
 // [tokens][heads][n_val][v_dim], n_val = kv heads (every value head) or 1 (the head's own); see attention_sink_prefill.cu.
+// The same on tcgen05 for heads that are not mixed (attention_sink_prefill_tc.cu): head sizes of any multiple of 8, keys up to 192, values up
+// to 128; writes the gated, rounded result and the columns of ones
+int hb_attention_sink_prefill_tc_supported(int n_heads, int n_kv_heads, int head_dim, int v_dim);
+int hb_attention_sink_prefill_tc(const void* q, long long q_stride, long long n_tokens, const void* k_cache, const void* v_cache,
+                                 const int* page_table, int pt_width, const int* seq_start, const int* seq_pos0, void* out, long long out_stride,
+                                 int ones, const float* gate, long long ldg, int gate_per, int n_seqs, int q_blocks, int n_heads, int n_kv_heads,
+                                 int head_dim, int v_dim, float scale, int window, int chunk, const float* sink, int n_pages, int* error_flag,
+                                 void* stream);
+// Few tokens per sequence, one block per (token, key/value head, key range) (attention_group.cu); supported: blocks per SM, 0: not built
+int hb_attention_group_supported(int n_heads, int n_kv_heads, int head_dim, int v_dim, int v_in_k);
+int hb_attention_group(const void* q, long long ldq, const void* k_cache, const void* v_cache, int v_in_k, const int* page_table, int pt_width,
+                       const int* tok_seq, const int* positions, float* scratch, void* out, int out_dtype, long long ldo, int ones,
+                       const float* gate, long long ldg, int gate_per, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int v_dim,
+                       float scale, int window, int chunk, const float* sink, int splits, int n_pages, int* status, void* stream);
 int hb_attention_sink_prefill_supported(int n_heads, int n_kv_heads, int head_dim, int v_dim);
 int hb_attention_sink_prefill(const void* q, long long q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                               int pt_width, const int* seq_start, const int* seq_pos0, float* out, int n_seqs, int q_blocks,
@@ -237,6 +251,12 @@ int hb_moe_glu(const void* h, int h_dtype, long long ldh, const void* w_gate, co
 int hb_moe_down(const void* act, int act_dtype, long long lda, const void* w_down, int w_dtype, const int* offsets, const int* order,
                 const int* tiles, int max_tiles, int top, float* down, long long ldd, int width, int ff, int tensor_cores, void* stream);
 // experts non-null: entries whose expert number is n_real or more are identity experts (their result is the row of h)
+// The two products on tcgen05 over plan tiles of 128 rows (moe_tc.cu): the inputs in the plan's order, then unit 0 (second product) or 1 to 3
+int hb_moe_gather(const void* h, long long ldh, const int* offsets, int n_experts, const int* order, int top, void* rows, int n_entries, int width,
+                  void* stream);
+int hb_moe_tc(const void* a, int n_entries, const void* w0, const void* w1, int n_experts, const int* offsets, const int* order, const int* tiles,
+              int max_tiles, int unit, void* out, long long ldo, int N, int K, float limit, float alpha, const float* in_weights, int sms,
+              int* error_flag, void* stream);
 int hb_moe_combine(const float* down, long long ldd, const float* weights, int top, float* out, long long ldo, int n_tokens, int width,
                    int accumulate, const int* experts, int n_real, const void* h, int h_dtype, long long ldh, void* stream);
 int hb_glu_clamp(const float* in, long long ldi, void* out, int out_dtype, long long ldo, int n_rows, int F, float limit, float alpha,

@@ -33,6 +33,7 @@
 #include "api.h"
 #include "common.cuh"
 #include "mma.cuh"
+#include "moe_act.cuh"
 
 #define MOE_BM 32
 #define MOE_BN 32
@@ -276,7 +277,7 @@ extern "C" int hb_moe_tile_rows(int tensor_cores) { return tensor_cores ? MM_BM 
 extern "C" int hb_moe_plan(const int* experts, int n_entries, int n_experts, int tile_rows, int* offsets, int* order, int* tiles, void* stream) {
     if (n_entries == 0) return 0;
     HB_REQUIRE(n_entries > 0 && n_experts > 0 && n_experts <= 4096, "moe_plan: bad sizes");
-    HB_REQUIRE(tile_rows == MOE_BM || tile_rows == MM_BM, "moe_plan: tiles of %d rows (%d or %d are built)", tile_rows, MOE_BM, MM_BM);
+    HB_REQUIRE(tile_rows == MOE_BM || tile_rows == MM_BM || tile_rows == 128, "moe_plan: tiles of %d rows (%d, %d or 128 are built)", tile_rows, MOE_BM, MM_BM);
     hb_launch(moe_plan_kernel, dim3(1), dim3(1024), sizeof(int) * 2 * n_experts, (cudaStream_t)stream, experts, n_entries, n_experts, tile_rows,
               offsets, order, tiles);
     return hb_check_launch("moe_plan");
@@ -285,22 +286,6 @@ extern "C" int hb_moe_plan(const int* experts, int n_entries, int n_experts, int
 extern "C" int hb_moe_max_tiles(int n_entries, int n_experts, int tile_rows) { return (n_entries + tile_rows - 1) / tile_rows + n_experts; }
 
 // ------------------------------------------------------------------------------------------------ the experts' products
-__device__ __forceinline__ float moe_gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
-// the first product's epilogue: the clamped gated unit of two matrices (MODE 1), the exact gelu of one (MODE 2), or the plain
-// silu-gated unit of two (MODE 3)
-template <int MODE>
-__device__ __forceinline__ float moe_first_act(float a0, float a1, float limit, float alpha);
-__device__ __forceinline__ float moe_glu(float g, float u, float limit, float alpha);
-template <> __device__ __forceinline__ float moe_first_act<1>(float a0, float a1, float limit, float alpha) { return moe_glu(a0, a1, limit, alpha); }
-template <> __device__ __forceinline__ float moe_first_act<2>(float a0, float a1, float limit, float alpha) { return moe_gelu_erf(a0); }
-template <> __device__ __forceinline__ float moe_first_act<3>(float a0, float a1, float limit, float alpha) { return silu_f32(a0) * a1; }
-template <> __device__ __forceinline__ float moe_first_act<0>(float a0, float a1, float limit, float alpha) { return a0; }
-__device__ __forceinline__ float moe_glu(float g, float u, float limit, float alpha) {
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return g * (1.0f / (1.0f + expf(-alpha * g))) * (u + 1.0f);
-}
-
 // GLU: a rows are h[token of the entry], two weight matrices [E][N][K], result act[slot][N] in TO.
 // else: a rows are act[slot], one weight matrix, result down[entry][N] in 32-bit.
 template <typename TA, typename TW, typename TO, int MODE>

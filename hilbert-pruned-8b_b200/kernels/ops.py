@@ -44,6 +44,11 @@ _SIGNATURES = {
                            _c_int, _c_ptr, _c_ptr],
     "hb_attention_sink_prefill": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                                   _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
+    "hb_attention_sink_prefill_tc": [_c_ptr, _c_ll, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_int, _c_ptr, _c_ll,
+                                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
+                                     _c_ptr],
+    "hb_attention_group": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_ptr,
+                           _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_head_mix_splits": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_ptr],
     "hb_mlstm_scan": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_float, _c_float, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
                       _c_int, _c_int, _c_ptr],
@@ -112,6 +117,9 @@ _SIGNATURES = {
                    _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_int, _c_ptr],
     "hb_moe_down": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int,
                     _c_ptr],
+    "hb_moe_gather": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr],
+    "hb_moe_tc": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_float, _c_float,
+                  _c_ptr, _c_int, _c_ptr, _c_ptr],
     "hb_moe_combine": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ptr],
     "hb_moe_route_scores": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
                             _c_ptr],
@@ -168,6 +176,8 @@ def load_library():
         for name in ("hb_attention_decode_supported", "hb_attention_prefill_supported", "hb_attention_prefill_tc_supported"):
             getattr(lib, name).argtypes, getattr(lib, name).restype = [_c_int, _c_int, _c_int], _c_int
         lib.hb_attention_sink_prefill_supported.argtypes, lib.hb_attention_sink_prefill_supported.restype = [_c_int] * 4, _c_int
+        lib.hb_attention_sink_prefill_tc_supported.argtypes, lib.hb_attention_sink_prefill_tc_supported.restype = [_c_int] * 4, _c_int
+        lib.hb_attention_group_supported.argtypes, lib.hb_attention_group_supported.restype = [_c_int] * 5, _c_int
         lib.hb_attention_heads_variant.argtypes, lib.hb_attention_heads_variant.restype = [_c_int] * 6, _c_int
         lib.hb_attention_heads_writes_output.argtypes, lib.hb_attention_heads_writes_output.restype = [_c_int] * 6, _c_int
         lib.hb_attention_pool_supported.argtypes, lib.hb_attention_pool_supported.restype = [_c_int] * 2, _c_int
@@ -330,6 +340,9 @@ class Ops:
         # terms) where the sizes allow; tests switch it off to compare with the FP32-pipe variant
         self.use_mma_attention = True
         self.use_flash_sink_attention = True    # steps of many tokens: attention_sink_prefill where it is built
+        self.use_tcgen05_sink_attention = True  # and on tcgen05 (attention_sink_prefill_tc) where heads are not mixed
+        self.use_tcgen05_experts = True         # experts' products of many rows on tcgen05 (moe_tc); tests compare both
+        self.use_group_attention = True         # steps of few tokens whose heads are not mixed: attention_group where it is built
         self.use_mma_pool_attention = True      # steps of many tokens: attention_pool_prefill where it is built (tests compare both)
         # Decode attention that rotates the new queries and key and appends to the cache itself
         # (no rotation kernel in front; the new key and value go into the owning split's copy of
@@ -657,6 +670,71 @@ class Ops:
                    int(chunk), self._f32_vec(sink, heads, "sink") if sink is not None else None,
                    cache.k.shape[0], self.status.data_ptr(), self._stream())
         self.launches += 1
+
+    def attention_sink_prefill_tc_wanted(self, step, heads: int, kv_heads: int, head_dim: int, v_dim: int, dtype) -> bool:
+        """Whether ``attention_sink_prefill_tc`` takes this step: as ``attention_sink_prefill_wanted``, 128 query tokens to a block."""
+        return bool(self.use_flash_sink_attention and self.use_tcgen05_sink_attention and dtype == torch.bfloat16 and not step.is_decode
+                    and step.max_new >= self.SINK_PREFILL_FROM
+                    and self.lib.hb_attention_sink_prefill_tc_supported(heads, kv_heads, head_dim, v_dim)
+                    and sum((n + 127) // 128 for n in step.host_new) <= 65535)
+
+    def attention_sink_prefill_tc(self, q, heads: int, kv_heads: int, head_dim: int, v_dim: int, cache, step, out, scale: float,
+                                  window: Optional[int], ones: int = 0, gate=None, chunk: int = 0, sink=None) -> None:
+        """``attention_sink`` on tcgen05, 128 query tokens of a sequence per block, no kept first tokens: ``out`` bfloat16 ``[tokens, heads *
+        v_dim + ones]``, normalised, times ``sigmoid(gate)`` (float32 ``[tokens, heads]`` or ``[tokens, heads * v_dim]``), then a one and zeros."""
+        self._dev(q, cache.k, cache.v, out, gate)
+        T = q.shape[0]
+        if any(t.dtype != torch.bfloat16 for t in (q, cache.k, cache.v, out)) or tuple(out.shape) != (T, heads * v_dim + ones) \
+                or tuple(q.shape) != (T, heads * head_dim) or not cache.k.is_contiguous() or not cache.v.is_contiguous():
+            raise KernelError("attention_sink_prefill_tc: bfloat16 queries, cache and output [tokens, heads * v_dim + ones] expected")
+        if tuple(cache.k.shape[1:]) != (kv_heads, 64, head_dim) or tuple(cache.v.shape[1:]) != (kv_heads, 64, v_dim):
+            raise KernelError("attention_sink_prefill_tc: cache layer does not match the heads")
+        pt = step.page_tables[cache.group]
+        q_blocks = sum((n + 127) // 128 for n in step.host_new)
+        self._call("hb_attention_sink_prefill_tc", q.data_ptr(), _rows(q, "queries"), T, cache.k.data_ptr(), cache.v.data_ptr(), pt.data_ptr(),
+                   pt.shape[1], step.seq_start.data_ptr(), step.seq_pos0.data_ptr(), out.data_ptr(), _rows(out, "attention output"), int(ones),
+                   *self._result_gate(gate, T, heads, v_dim), step.num_seqs, q_blocks, heads, kv_heads, head_dim, v_dim, float(scale),
+                   int(window) if window and not chunk else 0, int(chunk), self._f32_vec(sink, heads, "sink") if sink is not None else None,
+                   cache.k.shape[0], self.error_flag.data_ptr(), self._stream())
+        self.launches += 1
+
+    def attention_group_plan(self, tokens: int, heads: int, kv_heads: int, head_dim: int, v_dim: int, dtype, longest: int,
+                             values_in_keys: bool = False):
+        """How ``attention_group`` would run a step, or None when it is not built for these sizes: ``(splits, scratch)``, the key
+        ranges (whole pages; as many as fill the device once) and the floats of scratch that any step of these sizes needs."""
+        if not self.use_group_attention or dtype != torch.bfloat16 or tokens > 65535:
+            return None
+        blocks = int(self.lib.hb_attention_group_supported(heads, kv_heads, head_dim, v_dim, 1 if values_in_keys else 0))
+        if not blocks:
+            return None
+        group = heads // kv_heads
+        rows = 16 if group <= 16 else 32                     # query heads per block
+        units, target = tokens * kv_heads * -(-group // rows), self.sm_count * blocks
+        splits = max(1, min(target // units, (longest + 63) // 64, 64))
+        return splits, target * rows * (v_dim + 2)
+
+    def attention_group(self, q, heads: int, kv_heads: int, head_dim: int, v_dim: int, cache, step, out, scale: float, window: Optional[int],
+                        splits: int, scratch, ones: int = 0, gate=None, chunk: int = 0, sink=None, values_in_keys: bool = False) -> None:
+        """``attention_sink`` with one block per (token, key/value head, key range), no kept first tokens: ``out`` bfloat16 or float32
+        ``[tokens, heads * v_dim + ones]``, normalised, times ``sigmoid(gate)``, then a one and zeros.  ``values_in_keys``: a value row is the
+        first ``v_dim`` numbers of its key row; the value cache is not read.  ``scratch`` float32, for more than one key range."""
+        self._dev(q, cache.k, cache.v, out, gate, scratch)
+        T = q.shape[0]
+        if q.dtype != torch.bfloat16 or cache.k.dtype != torch.bfloat16 or tuple(q.shape) != (T, heads * head_dim) \
+                or tuple(out.shape) != (T, heads * v_dim + ones) or not cache.k.is_contiguous() or not cache.v.is_contiguous():
+            raise KernelError("attention_group: bfloat16 queries and cache and an output [tokens, heads * v_dim + ones] expected")
+        if tuple(cache.k.shape[1:]) != (kv_heads, 64, head_dim) or (not values_in_keys and tuple(cache.v.shape[1:]) != (kv_heads, 64, v_dim)):
+            raise KernelError("attention_group: cache layer does not match the heads")
+        if splits > 1 and (scratch is None or scratch.dtype != torch.float32 or scratch.numel() < T * heads * splits * (v_dim + 2)):
+            raise KernelError("attention_group: scratch of tokens * heads * splits * (v_dim + 2) floats expected")
+        pt = step.page_tables[cache.group]
+        self._call("hb_attention_group", q.data_ptr(), _rows(q, "queries"), cache.k.data_ptr(), cache.v.data_ptr(), 1 if values_in_keys else 0,
+                   pt.data_ptr(), pt.shape[1], step.tok_seq.data_ptr(), step.positions.data_ptr(), scratch.data_ptr() if scratch is not None else None,
+                   out.data_ptr(), _code(out), _rows(out, "attention output"), int(ones), *self._result_gate(gate, T, heads, v_dim), T, heads,
+                   kv_heads, head_dim, v_dim, float(scale), int(window) if window and not chunk else 0, int(chunk),
+                   self._f32_vec(sink, heads, "sink") if sink is not None else None, int(splits), cache.k.shape[0], self.status.data_ptr(),
+                   self._stream())
+        self.launches += 1 if splits == 1 else 2
 
     ATTENTION_HEADS_MAX_ROWS = 512      # tokens x key splits of a step that has fewer tokens than the device has SMs
 
@@ -1625,12 +1703,15 @@ class Ops:
     def moe_max_tiles(self, entries: int, n_experts: int, tile_rows: int) -> int:
         return int(self.lib.hb_moe_max_tiles(int(entries), int(n_experts), int(tile_rows)))
 
+    MOE_TC_ROWS = 24                # steps with so many entries per expert (on average) run the experts' products on tcgen05
+
     def moe_experts(self, h, experts, weights, w_gate, w_up, w_down, limit: float, alpha: float, out, accumulate: bool, workspace,
                     cap: int, tag: str = "", identity: bool = False, unit: str = "clamped_glu", weigh: str = "output"):
         """``out (+)= sum_k weights[t, k] * expert_{experts[t, k]}(h[t])`` with the experts' weights stacked ``[experts, ff,
         width]`` (gate, up) and ``[experts, width, ff]`` (down) in the activations' dtype and the clamped gated unit of
-        ``glu_clamp`` between them.  Four launches: plan, gate/up with activation, down, weighted sum.  bfloat16 operands whose
-        rows are multiples of 8 elements run the products on the tensor cores (``use_tensor_cores``), all others on the FP32 pipe.
+        ``glu_clamp`` between them.  Four or five launches: plan, (gathered inputs,) gate/up with activation, down, weighted sum.
+        bfloat16 operands whose rows are multiples of 8 elements run the products on the tensor cores (``use_tensor_cores``; tcgen05 for
+        ``MOE_TC_ROWS`` entries per expert or more, else mma.sync), all others on the FP32 pipe.
         ``w_up`` None: experts of one matrix, ``act = gelu_erf(w_gate h)`` (``limit`` and ``alpha`` unused).  ``identity``: expert
         numbers from the stack's size on are identity experts, whose result is ``h[t]`` itself.  ``unit`` "silu_glu": ``silu(gate) * up``
         between the products.  ``weigh`` "input": an expert is fed ``weights[t, k] * h[t]`` and its result is added as it is.
@@ -1652,7 +1733,9 @@ class Ops:
         most = cap * top
         tc = 1 if (self.use_tensor_cores and h.dtype == torch.bfloat16 and W % 8 == 0 and F % 8 == 0 and _rows(h, "expert input") % 8 == 0
                    and h.data_ptr() % 16 == 0) else 0
-        tile_rows = int(self.lib.hb_moe_tile_rows(tc))
+        # many rows per expert: tcgen05 over tiles of 128 rows; fewer: mma.sync over tiles of 64 (or the FP32 pipe over tiles of 32)
+        umma = bool(tc and self.use_tcgen05_experts and entries >= self.MOE_TC_ROWS * E)
+        tile_rows = 128 if umma else int(self.lib.hb_moe_tile_rows(tc))
         max_tiles = self.moe_max_tiles(entries, E, tile_rows)
         plan = workspace.buffer("moe.plan" + tag, (E + 1 + most + 1 + 2 * self.moe_max_tiles(most, E, 32),), torch.int32)
         offsets, order, tiles = plan[: E + 1], plan[E + 1: E + 1 + most], plan[E + 1 + most:]
@@ -1660,14 +1743,25 @@ class Ops:
         down = workspace.buffer("moe.down" + tag, (most, W), torch.float32)
         s = self._stream()
         self._call("hb_moe_plan", experts.data_ptr(), entries, E, tile_rows, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), s)
-        self._call("hb_moe_glu", h.data_ptr(), _code(h), _rows(h, "expert input"), w_gate.data_ptr(),
-                   w_up.data_ptr() if w_up is not None else None, _code(w_gate),
-                   offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles, top, act.data_ptr(), _code(act), F, F, W,
-                   2 if w_up is None else {"clamped_glu": 1, "silu_glu": 3}[unit], float(limit), float(alpha),
-                   weights.data_ptr() if weigh == "input" else None, tc, s)
-        self._call("hb_moe_down", act.data_ptr(), _code(act), F, w_down.data_ptr(), _code(w_down), offsets.data_ptr(), order.data_ptr(),
-                   tiles.data_ptr(), max_tiles, top, down.data_ptr(), W, W, F, tc, s)
-        self.launches += 3
+        unit_code = 2 if w_up is None else {"clamped_glu": 1, "silu_glu": 3}[unit]
+        in_weights = weights.data_ptr() if weigh == "input" else None
+        if umma:
+            rows = workspace.buffer("moe.rows" + tag, (most, W), h.dtype)
+            self._call("hb_moe_gather", h.data_ptr(), _rows(h, "expert input"), offsets.data_ptr(), E, order.data_ptr(), top, rows.data_ptr(), entries, W, s)
+            self._call("hb_moe_tc", rows.data_ptr(), entries, w_gate.data_ptr(), w_up.data_ptr() if w_up is not None else None, E, offsets.data_ptr(),
+                       order.data_ptr(), tiles.data_ptr(), max_tiles, unit_code, act.data_ptr(), F, F, W, float(limit), float(alpha), in_weights,
+                       self.sm_count, self.error_flag.data_ptr(), s)
+            self._call("hb_moe_tc", act.data_ptr(), entries, w_down.data_ptr(), None, E, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles,
+                       0, down.data_ptr(), W, W, F, 0.0, 0.0, None, self.sm_count, self.error_flag.data_ptr(), s)
+            self.launches += 4
+        else:
+            self._call("hb_moe_glu", h.data_ptr(), _code(h), _rows(h, "expert input"), w_gate.data_ptr(),
+                       w_up.data_ptr() if w_up is not None else None, _code(w_gate),
+                       offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles, top, act.data_ptr(), _code(act), F, F, W,
+                       unit_code, float(limit), float(alpha), in_weights, tc, s)
+            self._call("hb_moe_down", act.data_ptr(), _code(act), F, w_down.data_ptr(), _code(w_down), offsets.data_ptr(), order.data_ptr(),
+                       tiles.data_ptr(), max_tiles, top, down.data_ptr(), W, W, F, tc, s)
+            self.launches += 3
         if out is None:
             return down[:entries]
         self._call("hb_moe_combine", down.data_ptr(), W, weights.data_ptr() if weigh == "output" else None, top, out.data_ptr(), _rows(out, "expert output"), T, W,

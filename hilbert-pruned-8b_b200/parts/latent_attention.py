@@ -68,9 +68,10 @@ class LatentAttention(Mixer):
         self.gate_at = self.down_at + (0 if self.shares_cache else self.rank + self.dr)
         self.guest_at = None
         self.key_dim = self.rank + self.dr
-        # head sizes of the written-out form (multiples of 64, as the prompt kernel wants them)
-        self.flat_d = (self.d + self.dr + 63) // 64 * 64
-        self.flat_dv = (self.dv + 63) // 64 * 64
+        # head sizes of the written-out form, as the prompt kernels want them: multiples of 8 for tcgen05, beyond its sizes of 64
+        to = 8 if self.d + self.dr <= 192 and self.dv <= 128 else 64
+        self.flat_d = (self.d + self.dr + to - 1) // to * to
+        self.flat_dv = (self.dv + to - 1) // to * to
         self.write_out = True                 # tests switch it off to run every step in the folded form
         self.w_in = self.w_uk = self.w_uv = self.w_o = self.c_weight = self.w_ukv = self.w_o_flat = self.w_uq = self.q_weight = None
 
@@ -154,15 +155,18 @@ class LatentAttention(Mixer):
         ops.latent_prepare(q_raw, down, H, d, dr, rank, self.c_weight, self.eps, table, rot, q, cache, step, append)
         ops.head_linear(q_raw, d + dr, self.w_uk, q, self.key_dim, d, rank)
         mixed = ws.buffer("latent_attention.mixed", (cap, H * rank), torch.float32)[:T]
-        softmax_attention(self.ctx, q, H, 1, self.key_dim, rank, cache, step, self.scale, self.window, 0, mixed, sink=self.sink_logits)
+        softmax_attention(self.ctx, q, H, 1, self.key_dim, rank, cache, step, self.scale, self.window, 0, mixed, sink=self.sink_logits,
+                          values_in_keys=True)
         attn = ws.buffer("latent_attention.out", (cap, H * dv), self.ctx.dtype)[:T]
         ops.head_linear(mixed, rank, self.w_uv, attn, dv, rank, dv, gate=gate)
         ops.linear(attn, self.w_o, residual, accumulate=accumulate)
 
     def written_out(self, step) -> bool:
         """Whether this step writes every head's keys and values out and runs the tensor-core prompt kernel on them."""
-        return bool(self.write_out and self.ctx.dtype == torch.bfloat16 and self.ctx.ops.attention_sink_prefill_wanted(
-            step, self.heads, self.heads, self.flat_d, self.flat_dv, self.ctx.dtype))
+        sizes = (step, self.heads, self.heads, self.flat_d, self.flat_dv, self.ctx.dtype)
+        ops = self.ctx.ops
+        return bool(self.write_out and self.ctx.dtype == torch.bfloat16
+                    and (ops.attention_sink_prefill_tc_wanted(*sizes) or ops.attention_sink_prefill_wanted(*sizes)))
 
     def _forward_written_out(self, q_raw, down, table, rot, gate, residual, step, cache, append: bool, accumulate: bool) -> None:
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens

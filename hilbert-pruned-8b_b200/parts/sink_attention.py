@@ -183,16 +183,34 @@ class SinkAttention(Mixer):
 
 
 def softmax_attention(ctx, q, H: int, G: int, d: int, dv: int, cache, step, scale: float, window: Optional[int], keep_first: int, out,
-                      ones: int = 0, gate=None, talk_matrix=None, use_heads_kernel: bool = True, chunk: int = 0, sink=None) -> None:
+                      ones: int = 0, gate=None, talk_matrix=None, use_heads_kernel: bool = True, chunk: int = 0, sink=None,
+                      values_in_keys: bool = False) -> None:
     """Softmax attention of the step's queries ``q [tokens, H * d]`` over the cached keys and values of ``cache`` (``G``
     key/value heads of sizes ``d`` and ``dv``), by whichever kernel takes the step: ``out [tokens, H * dv + ones]`` (the
     dtype of the products, or 32-bit) receives the normalised results, mixed between the heads by ``talk_matrix``, each
     head's times ``sigmoid(gate[t, head])`` (``gate`` ``[tokens, H * dv]``: every element's times its own), and ``ones`` more columns (a one, then zeros).  ``chunk`` (instead of a window) and
-    ``sink`` (float32 ``[H]``) as the kernels take them.  Any part that has put its keys
+    ``sink`` (float32 ``[H]``) as the kernels take them.  ``values_in_keys``: a value row is the first ``dv`` numbers of its key row, and a
+    kernel that knows it reads the key rows only.  Any part that has put its keys
     and values into a paged cache group can call it."""
     ops, ws, T, cap = ctx.ops, ctx.workspace, step.num_tokens, ctx.max_step_tokens
     talk = talk_matrix is not None
     longest = min(step.max_len, chunk) if chunk else step.max_len if window is None else min(step.max_len, window + keep_first)
+    plain = use_heads_kernel and not talk and not keep_first       # every head its own weights, one run of visible keys
+    if plain and out.dtype == torch.bfloat16 and ops.attention_sink_prefill_tc_wanted(step, H, G, d, dv, ctx.dtype) \
+            and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0:
+        # many tokens: 128 query tokens of a sequence per block, on tcgen05
+        ops.attention_sink_prefill_tc(q, H, G, d, dv, cache, step, out, scale, window, ones=ones, gate=gate, chunk=chunk, sink=sink)
+        return
+    few = None
+    if plain and not ops.attention_sink_prefill_wanted(step, H, G, d, dv, ctx.dtype):
+        few = ops.attention_group_plan(T, H, G, d, dv, ctx.dtype, longest, values_in_keys)
+    if few is not None and q.data_ptr() % 16 == 0:
+        # few tokens: one block per (token, key/value head, key range) serves the head's group of query heads
+        splits, floats = few
+        scratch = ws.buffer(f"attention_group.{H}.{G}.{dv}", (floats,), torch.float32)
+        ops.attention_group(q, H, G, d, dv, cache, step, out, scale, window, splits, scratch, ones=ones, gate=gate, chunk=chunk, sink=sink,
+                            values_in_keys=values_in_keys)
+        return
     plan = ops.attention_heads_plan(T, H, G, d, dv, ctx.dtype, longest) if use_heads_kernel else None
     if use_heads_kernel and ops.attention_sink_prefill_wanted(step, H, G, d, dv, ctx.dtype):
         # many tokens: 64 query tokens of a sequence share a block's keys and values (flash-style, tensor cores)

@@ -432,7 +432,7 @@ def test_chunked_attention_with_probes_at_the_edges_and_a_sink(dtype):
         for sizes in ((300,), (60, 3, 1, 1, 1, 1, 1, 1, 1, 58, 1, 1, 1, 1, 1, 1, 1, 300), (2, 126, 1, 1, 300)):
             run = _MixerRun(c, spec, w)
             _close(run.feed(hs, sizes), want, dtype, f"chunk attention {(H, G, d, chunk, rot)} portions {sizes}")
-        for flag in ("use_mma_attention", "use_flash_sink_attention"):      # the other kernels for the same steps
+        for flag in ("use_tcgen05_sink_attention", "use_group_attention", "use_mma_attention", "use_flash_sink_attention"):      # the other kernels for the same steps
             setattr(c.ops, flag, False)
             _close(_MixerRun(c, spec, w).feed(hs, (150, 1, 1, 300)), want, dtype, f"chunk attention {(H, G, d, chunk, rot)} without {flag}")
         run = _MixerRun(c, spec, w)
