@@ -38,9 +38,10 @@ int hb_gemm_tc_token_tile(int M);
 long long hb_gemm_tc_scratch_floats(int M, int N, int K, int mode, int schedule);
 long long hb_gemm_tc_tiles(int M, int N, int mode);
 int hb_gemm_tc_resident_clusters(int mode, int size);
+// (mode 3, the gated units: unit_alpha 0: silu(g) u; else the clamped unit with unit_limit)
 int hb_gemm_tc(const void* a, long long lda, const void* w, long long ldw, long long w_rows, void* out, long long ldc,
                int M, int N, int K, int mode, int up_row0, int schedule, float* partials, long long partials_capacity,
-               int* tile_counters, long long counters_capacity, int* error_flag, int packed, void* stream);
+               int* tile_counters, long long counters_capacity, int* error_flag, int packed, float unit_alpha, float unit_limit, void* stream);
 // A norm between two products, folded into them (hb_gemm_tc_fold; null pointers: that side is not used).
 typedef struct {
     const float* prep_w;        // producer (mode 2): the norm's weight; the factor is prep_offset + prep_w[feature]
@@ -56,11 +57,12 @@ typedef struct {
 } HbNormFold;
 int hb_gemm_tc_fold(const void* a, long long lda, const void* w, long long ldw, long long w_rows, void* out, long long ldc,
                int M, int N, int K, int mode, int up_row0, int schedule, float* partials, long long partials_capacity,
-               int* tile_counters, long long counters_capacity, int* error_flag, int packed, const HbNormFold* fold, void* stream);
+               int* tile_counters, long long counters_capacity, int* error_flag, int packed, float unit_alpha, float unit_limit,
+               const HbNormFold* fold, void* stream);
 int hb_gemm_tc2_wanted(int M, int N, int K);
 int hb_gemm_tc2_resident_pairs(int mode);
 int hb_gemm_tc2(const void* a, long long lda, const void* w, long long ldw, long long w_rows, void* out, long long ldc,
-                int M, int N, int K, int mode, int up_row0, int* error_flag, int packed, void* stream);
+                int M, int N, int K, int mode, int up_row0, int* error_flag, int packed, float unit_alpha, float unit_limit, void* stream);
 int hb_attention_general(const void* q, int q_dtype, long long q_stride, const void* k_cache, const void* v_cache,
                          int cache_dtype, const int* page_table, int pt_width, const int* tok_seq,
                          const int* positions, void* out, int out_dtype, long long out_stride, int n_tokens,

@@ -113,6 +113,60 @@ qkv_prepare_kernel(const TP* __restrict__ proj, long long ldp, const float* __re
     }
 }
 
+// The same without norm, rotation and value mixing, where rows and heads are whole pieces of four numbers: bias, rounding, queries to
+// their buffer, keys and values into the cache, a token's pieces to a block.
+#define QR_THREADS 256
+template <typename TQ>
+__device__ __forceinline__ void qr_store(TQ* p, const float4 v) {
+    if constexpr (sizeof(TQ) == 2) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        uint2 pk;
+        pk.x = *reinterpret_cast<uint32_t*>(&lo);
+        pk.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(p) = pk;
+    } else {
+        *reinterpret_cast<float4*>(p) = v;
+    }
+}
+
+template <typename TQ>
+__global__ void __launch_bounds__(QR_THREADS)
+qkv_rows_kernel(const float* __restrict__ proj, long long ldp, const float* __restrict__ bias, int nh, int nkv, int hd, int vd, TQ* __restrict__ q_out,
+                long long ldq, TQ* __restrict__ k_cache, TQ* __restrict__ v_cache, const int* __restrict__ page_table, int pt_width,
+                const int* __restrict__ tok_seq, const int* __restrict__ positions, int n_pages, int append, int* status) {
+    pdl_trigger();
+    const int t = blockIdx.x;
+    int page = -1, pos = 0;
+    if (append) {
+        pos = positions[t];
+        const int lp = pos / HB_PAGE_TOKENS;
+        page = lp < pt_width ? page_table[(size_t)tok_seq[t] * pt_width + lp] : -1;
+        if (page < 0 || page >= n_pages) {
+            if (threadIdx.x == 0 && blockIdx.y == 0) hb_note(status, HB_STATUS_PAGE, 1 + tok_seq[t]);
+            page = -1;
+        }
+    }
+    pdl_wait();
+    proj = pdl_fresh(proj);
+    const float* row = proj + (size_t)t * ldp;
+    const int q_end = nh * hd, k_end = q_end + nkv * hd, all = page >= 0 ? k_end + nkv * vd : q_end;
+    for (int c = (blockIdx.y * QR_THREADS + threadIdx.x) * 4; c < all; c += gridDim.y * QR_THREADS * 4) {
+        float4 x = *reinterpret_cast<const float4*>(row + c);
+        if (bias != nullptr) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + c);
+            x = make_float4(x.x + b.x, x.y + b.y, x.z + b.z, x.w + b.w);
+        }
+        if (c < q_end) qr_store<TQ>(q_out + (size_t)t * ldq + c, x);
+        else if (c < k_end) {
+            const int u = c - q_end, g = u / hd;
+            qr_store<TQ>(k_cache + cache_offset(page, g, pos, nkv, hd) + (u - g * hd), x);
+        } else {
+            const int u = c - k_end, g = u / vd;
+            qr_store<TQ>(v_cache + cache_offset(page, g, pos, nkv, vd) + (u - g * vd), x);
+        }
+    }
+}
+
 extern "C" int hb_qkv_prepare(const void* proj, int proj_dtype, long long ldp, const float* bias, const float* table, int rot,
                               int n_heads, int n_kv_heads, int head_dim, int v_dim, int unit_norm, const float* q_norm_w,
                               const float* k_norm_w, float eps, void* q_out, int q_dtype, long long ldq, void* k_cache, void* v_cache, int cache_dtype, const int* page_table,
@@ -132,8 +186,22 @@ extern "C" int hb_qkv_prepare(const void* proj, int proj_dtype, long long ldp, c
     HB_REQUIRE(n_heads + 2 * n_kv_heads <= 65535, "qkv_prepare: too many heads");
     const bool cache_same = (q_dtype == cache_dtype);
     HB_REQUIRE(cache_same, "qkv_prepare: queries and cache must have one dtype");
-    dim3 grid(n_tokens, n_heads + (append ? 2 * n_kv_heads : 0));
     cudaStream_t s = (cudaStream_t)stream;
+    const int qe = q_dtype == HB_BF16 ? 2 : 4;
+    if (proj_dtype == HB_F32 && (q_dtype == HB_BF16 || q_dtype == HB_F32) && unit_norm == 0 && rot == 0 && v_mode == 0 && !v_from_k &&
+        ((head_dim | v_dim) & 3) == 0 && (ldp & 3) == 0 && (ldq & 3) == 0 && (((uintptr_t)proj | (uintptr_t)bias) & 15) == 0 &&
+        (((uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & (qe * 4 - 1)) == 0) {
+        const int columns = n_heads * head_dim + (append ? n_kv_heads * (head_dim + v_dim) : 0);
+        dim3 rgrid(n_tokens, min(65535, (columns / 4 + 4 * QR_THREADS - 1) / (4 * QR_THREADS)));
+        if (q_dtype == HB_BF16)
+            hb_launch(qkv_rows_kernel<bf16>, dim3(rgrid), dim3(QR_THREADS), 0, s, (const float*)proj, ldp, bias, n_heads, n_kv_heads, head_dim, v_dim, (bf16*)q_out,
+                      ldq, (bf16*)k_cache, (bf16*)v_cache, page_table, pt_width, tok_seq, positions, n_pages, append, status);
+        else
+            hb_launch(qkv_rows_kernel<float>, dim3(rgrid), dim3(QR_THREADS), 0, s, (const float*)proj, ldp, bias, n_heads, n_kv_heads, head_dim, v_dim, (float*)q_out,
+                      ldq, (float*)k_cache, (float*)v_cache, page_table, pt_width, tok_seq, positions, n_pages, append, status);
+        return hb_check_launch("qkv_rows");
+    }
+    dim3 grid(n_tokens, n_heads + (append ? 2 * n_kv_heads : 0));
 #define HB_QP_LAUNCH(TP, TQ)                                                                                                   \
     hb_launch(qkv_prepare_kernel<TP, TQ, TQ>, dim3(grid), dim3(QP_THREADS), 0, s, (const TP*)proj, ldp, bias, (const float2*)table, rot,  \
               n_heads, n_kv_heads, head_dim, v_dim, unit_norm, q_norm_w, k_norm_w, eps, (TQ*)q_out, ldq, (TQ*)k_cache, (TQ*)v_cache, page_table,       \

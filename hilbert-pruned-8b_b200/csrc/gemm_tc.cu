@@ -256,7 +256,7 @@ static int dispatch_bn(int bn, bool cluster, int mode, const CUtensorMap& mw, co
 extern "C" int hb_gemm_tc_fold(const void* a, long long lda, const void* w, long long ldw, long long w_rows, void* out,
                                long long ldc, int M, int N, int K, int mode, int up_row0, int schedule, float* partials,
                                long long partials_capacity, int* tile_counters, long long counters_capacity, int* error_flag,
-                               int packed, const HbNormFold* fold, void* stream) {
+                               int packed, float unit_alpha, float unit_limit, const HbNormFold* fold, void* stream) {
     if (M == 0 || N == 0) return 0;
     HB_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
     HB_REQUIRE(mode >= 0 && mode <= 3, "gemm_tc: unknown epilogue %d", mode);
@@ -311,6 +311,8 @@ extern "C" int hb_gemm_tc_fold(const void* a, long long lda, const void* w, long
     prm.N = N;
     prm.K = K;
     prm.up_row0 = up_row0;
+    prm.unit_alpha = unit_alpha;
+    prm.unit_limit = unit_limit;
     prm.tiles_m = pl.tiles_m;
     prm.tiles_n = pl.tiles_n;
     prm.kb_total = pl.kb_total;
@@ -330,7 +332,7 @@ extern "C" int hb_gemm_tc_fold(const void* a, long long lda, const void* w, long
 extern "C" int hb_gemm_tc(const void* a, long long lda, const void* w, long long ldw, long long w_rows, void* out,
                           long long ldc, int M, int N, int K, int mode, int up_row0, int schedule, float* partials,
                           long long partials_capacity, int* tile_counters, long long counters_capacity, int* error_flag,
-                          int packed, void* stream) {
+                          int packed, float unit_alpha, float unit_limit, void* stream) {
     return hb_gemm_tc_fold(a, lda, w, ldw, w_rows, out, ldc, M, N, K, mode, up_row0, schedule, partials, partials_capacity, tile_counters,
-                           counters_capacity, error_flag, packed, nullptr, stream);
+                           counters_capacity, error_flag, packed, unit_alpha, unit_limit, nullptr, stream);
 }

@@ -292,7 +292,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
 #pragma unroll
                         for (int j = 0; j < 16; j++) {
                             const float other = theirs[j * 64 + f];
-                            const float y = gate_thread ? silu_fast(v[0][j]) * other : silu_fast(other) * v[1][j];
+                            const float y = gate_thread ? tc_unit(p, v[0][j], other) : tc_unit(p, other, v[1][j]);
                             yb[((gate_thread ? 0 : 16) + j) * 64 + f] = __float2bfloat16_rn(y);
                         }
                         fence_async_shared();
@@ -456,7 +456,8 @@ extern "C" int hb_gemm_tc2_wanted(int M, int N, int K) {
 
 // Arguments as hb_gemm_tc (no scratch: whole tiles only).
 extern "C" int hb_gemm_tc2(const void* a, long long lda, const void* w, long long ldw, long long w_rows, void* out,
-                           long long ldc, int M, int N, int K, int mode, int up_row0, int* error_flag, int packed, void* stream) {
+                           long long ldc, int M, int N, int K, int mode, int up_row0, int* error_flag, int packed, float unit_alpha,
+                           float unit_limit, void* stream) {
     if (M == 0 || N == 0) return 0;
     HB_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc2: bad sizes M=%d N=%d K=%d", M, N, K);
     HB_REQUIRE(mode >= 0 && mode <= 3, "gemm_tc2: unknown epilogue %d", mode);
@@ -480,6 +481,8 @@ extern "C" int hb_gemm_tc2(const void* a, long long lda, const void* w, long lon
     prm.N = N;
     prm.K = K;
     prm.up_row0 = up_row0;
+    prm.unit_alpha = unit_alpha;
+    prm.unit_limit = unit_limit;
     prm.tiles_m = (M + T2_TOKENS - 1) / T2_TOKENS;
     prm.tiles_n = (N + 2 * feat - 1) / (2 * feat);
     prm.kb_total = (K + TC_BK - 1) / TC_BK;

@@ -8,7 +8,8 @@
 //  * latent_prepare: per token, the latent part of the down projection divided by its root mean
 //    square and multiplied by a weight, the shared key part turned by the step's rotation table, both
 //    written to the cache (key row [c | k_r], value row c); every head's rotated query part turned
-//    and written behind the place of its q'.  The rotation pairs dimensions (2i, 2i + 1).
+//    and written behind the place of its q'.  The rotation pairs dimensions (2i, 2i + 1).  Queries of
+//    whole pieces of four numbers go through latent_queries, a token's pieces to a block.
 //  * latent_gather, latent_scatter: keys and values of every head written out for steps of many tokens (see there).
 //  * head_linear: out[t, h, :] = W_h in[t, h, :] for every head, W given as [heads][n_in][n_out]
 //    (the output index contiguous), 32-bit accumulation on the FP32 pipe; optionally times
@@ -24,10 +25,10 @@ latent_prepare_kernel(const float* __restrict__ q, long long ldq_in, const float
                       const float* __restrict__ c_weight, float eps, const float2* __restrict__ table, int rot,
                       TQ* __restrict__ q_out, long long ldq, int q_head, int q_rot_at, int q_copy, TQ* __restrict__ k_cache, TQ* __restrict__ v_cache,
                       const int* __restrict__ page_table, int pt_width, const int* __restrict__ tok_seq,
-                      const int* __restrict__ positions, int n_pages, int append, int* status) {
+                      const int* __restrict__ positions, int n_pages, int append, int slot0, int* status) {
     pdl_trigger();
     __shared__ float scratch[33];
-    const int t = blockIdx.x, slot = blockIdx.y, tid = threadIdx.x;
+    const int t = blockIdx.x, slot = slot0 + blockIdx.y, tid = threadIdx.x;
     const int pos = positions[t], half = rot >> 1;
     int page = -1;
     if (slot == nh) {
@@ -85,6 +86,55 @@ latent_prepare_kernel(const float* __restrict__ q, long long ldq_in, const float
     for (int i = rot + tid; i < dr; i += LP_THREADS) kr[rank + i] = from_f32<TQ>(src[rank + i]);
 }
 
+// The queries' part of the same where every run of a head is whole pieces of four numbers: a thread takes pieces of the token's
+// queries one after the other (32-bit pieces of 16 bytes in, pieces of the queries' dtype out), whatever head they are of.
+#define LQ_THREADS 256
+#define LQ_FROM 64             // (few tokens: one launch for queries and latents)
+template <typename TQ>
+__device__ __forceinline__ void lq_store(TQ* p, const float4 v) {
+    if constexpr (sizeof(TQ) == 2) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        uint2 pk;
+        pk.x = *reinterpret_cast<uint32_t*>(&lo);
+        pk.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(p) = pk;
+    } else {
+        *reinterpret_cast<float4*>(p) = v;
+    }
+}
+
+template <typename TQ>
+__global__ void __launch_bounds__(LQ_THREADS)
+latent_queries_kernel(const float* __restrict__ q, long long ldq_in, int nh, int d, int dr, const float4* __restrict__ table, int rot,
+                      TQ* __restrict__ q_out, long long ldq, int q_head, int q_rot_at, int q_copy) {
+    pdl_trigger();
+    pdl_wait();
+    q = pdl_fresh(q);
+    table = pdl_fresh(table);
+    const int t = blockIdx.x;
+    const float* row = q + (size_t)t * ldq_in;
+    TQ* orow = q_out + (size_t)t * ldq;
+    // pieces per head: [unrotated, copied, and the zeros behind the head, or neither | rotated]
+    const int first = q_copy > 0 ? 0 : q_rot_at, per = ((q_copy > 0 ? q_head : q_rot_at + dr) - first) >> 2;
+    for (int i = blockIdx.y * LQ_THREADS + threadIdx.x; i < nh * per; i += gridDim.y * LQ_THREADS) {
+        const int h = i / per, c = first + ((i - h * per) << 2), u = c - q_rot_at;      // u: the piece's place in the rotated part
+        const float* src = row + (size_t)h * (d + dr);
+        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (u < 0) x = *reinterpret_cast<const float4*>(src + c);
+        else if (u < dr) {
+            x = *reinterpret_cast<const float4*>(src + d + u);
+            if (u < rot) {
+                const float4 cs = table[((size_t)t * (rot >> 1) + (u >> 1)) >> 1];        // (cos, sin) of two neighbouring pairs
+                float4 y;
+                rope_pair(x.x, x.y, cs.x, cs.y, y.x, y.y);
+                rope_pair(x.z, x.w, cs.z, cs.w, y.z, y.w);
+                x = y;
+            }
+        }
+        lq_store<TQ>(orow + (size_t)h * q_head + c, x);
+    }
+}
+
 // q: the queries' projections [tokens][heads x (d + dr)]; down: [latent | shared key part] per token, needed only with `append`
 // (a layer that reads another layer's latents has none).
 extern "C" int hb_latent_prepare(const float* q, long long ldq_in, const float* down, long long ldd, int n_heads, int d, int dr, int rank,
@@ -99,17 +149,33 @@ extern "C" int hb_latent_prepare(const float* q, long long ldq_in, const float* 
     HB_REQUIRE(q_rot_at >= 0 && q_rot_at + dr <= q_head && (q_copy == 0 || (q_copy == d && q_rot_at == d)),
                "latent_prepare: the rotated part at %d of %d columns per head (%d copied) does not fit", q_rot_at, q_head, q_copy);
     HB_REQUIRE(q_dtype == cache_dtype, "latent_prepare: queries and cache must have one dtype");
-    dim3 grid(n_tokens, n_heads + (append ? 1 : 0));
     cudaStream_t s = (cudaStream_t)stream;
+    HB_REQUIRE(q_dtype == HB_BF16 || q_dtype == HB_F32, "latent_prepare: unsupported dtype %d", q_dtype);
+    int slot0 = 0;                                          // first of the general kernel's slots: the heads, then the latent
+    const int qe = q_dtype == HB_BF16 ? 2 : 4;
+    if (n_tokens >= LQ_FROM && ((d | dr | rot | q_head | q_rot_at) & 3) == 0 && (ldq_in & 3) == 0 && (ldq & 3) == 0 && (((uintptr_t)q | (uintptr_t)table) & 15) == 0 &&
+        ((uintptr_t)q_out & (qe * 4 - 1)) == 0 && (q_copy > 0 || dr > 0)) {
+        const int pieces = n_heads * (((q_copy > 0 ? q_head : q_rot_at + dr) - (q_copy > 0 ? 0 : q_rot_at)) / 4);
+        dim3 qgrid(n_tokens, min(65535, max(1, (pieces + 4 * LQ_THREADS - 1) / (4 * LQ_THREADS))));
+        if (q_dtype == HB_BF16)
+            hb_launch(latent_queries_kernel<bf16>, dim3(qgrid), dim3(LQ_THREADS), 0, s, q, ldq_in, n_heads, d, dr, (const float4*)table, rot, (bf16*)q_out, ldq,
+                      q_head, q_rot_at, q_copy);
+        else
+            hb_launch(latent_queries_kernel<float>, dim3(qgrid), dim3(LQ_THREADS), 0, s, q, ldq_in, n_heads, d, dr, (const float4*)table, rot, (float*)q_out, ldq,
+                      q_head, q_rot_at, q_copy);
+        if (hb_check_launch("latent_queries")) return 1;
+        if (!append) return 0;
+        slot0 = n_heads;
+    }
+    dim3 grid(n_tokens, n_heads + (append ? 1 : 0) - slot0);
     if (q_dtype == HB_BF16)
         hb_launch(latent_prepare_kernel<bf16>, dim3(grid), dim3(LP_THREADS), 0, s, q, ldq_in, down, ldd, n_heads, d, dr, rank, c_weight, eps,
                   (const float2*)table, rot, (bf16*)q_out, ldq, q_head, q_rot_at, q_copy, (bf16*)k_cache, (bf16*)v_cache, page_table, pt_width, tok_seq, positions,
-                  n_pages, append, status);
-    else if (q_dtype == HB_F32)
+                  n_pages, append, slot0, status);
+    else
         hb_launch(latent_prepare_kernel<float>, dim3(grid), dim3(LP_THREADS), 0, s, q, ldq_in, down, ldd, n_heads, d, dr, rank, c_weight, eps,
                   (const float2*)table, rot, (float*)q_out, ldq, q_head, q_rot_at, q_copy, (float*)k_cache, (float*)v_cache, page_table, pt_width, tok_seq, positions,
-                  n_pages, append, status);
-    else return hb_fail("latent_prepare: unsupported dtype %d", q_dtype);
+                  n_pages, append, slot0, status);
     return hb_check_launch("latent_prepare");
 }
 
@@ -190,6 +256,26 @@ latent_scatter_kernel(const bf16* __restrict__ kv, long long ldkv, const bf16* _
     const bf16* src = kv + (size_t)sp * HB_PAGE_TOKENS * ldkv;
     bf16* kd = k_out + ((size_t)sp * nh + h) * HB_PAGE_TOKENS * hd_out;
     bf16* vd = v_out + ((size_t)sp * nh + h) * HB_PAGE_TOKENS * vd_out;
+    if (((d | dr | dv | rank | hd_out | vd_out) & 7) == 0 && (ldkv & 7) == 0) {
+        // whole 16-byte pieces: a piece is part of one of [unrotated | rotated | zeros]
+        const uint4 zero8 = make_uint4(0u, 0u, 0u, 0u);
+        const int kp = hd_out >> 3, vp = vd_out >> 3;
+        for (int i = tid; i < HB_PAGE_TOKENS * kp; i += LE_THREADS) {
+            const int r = i / kp, c = (i - r * kp) << 3;
+            uint4 x = zero8;
+            if (r < valid) {
+                if (c < d) x = *reinterpret_cast<const uint4*>(src + (size_t)r * ldkv + (size_t)h * d + c);
+                else if (c < d + dr) x = *reinterpret_cast<const uint4*>(krot + (size_t)r * (rank + dr) + (c - d));
+            }
+            *reinterpret_cast<uint4*>(kd + (size_t)i * 8) = x;
+        }
+        for (int i = tid; i < HB_PAGE_TOKENS * vp; i += LE_THREADS) {
+            const int r = i / vp, c = (i - r * vp) << 3;
+            *reinterpret_cast<uint4*>(vd + (size_t)i * 8) =
+                (r < valid && c < dv) ? *reinterpret_cast<const uint4*>(src + (size_t)r * ldkv + (size_t)nh * d + (size_t)h * dv + c) : zero8;
+        }
+        return;
+    }
     for (int i = tid; i < HB_PAGE_TOKENS * hd_out; i += LE_THREADS) {
         const int r = i / hd_out, c = i - r * hd_out;
         bf16 x = zero;

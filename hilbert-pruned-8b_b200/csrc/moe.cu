@@ -47,35 +47,86 @@
 #define MM_THREADS 256
 
 // ------------------------------------------------------------------------------------------------ route
-template <typename TH>
-__global__ void __launch_bounds__(256)
+// One block: TOKENS tokens, whose rows are staged once, so that a row of the router's matrix serves all of them; a warp per
+// expert for the logits (four columns at a time where rows are 16-byte aligned: `vec`), a warp per token for the choice.
+#define MR_THREADS 512
+#define MR_WARPS (MR_THREADS / 32)
+
+__device__ __forceinline__ float4 mr_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 mr_load4(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename TH, int TOKENS>
+__global__ void __launch_bounds__(MR_THREADS)
 moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restrict__ wr, const float* __restrict__ bias,
-                 int* __restrict__ experts, float* __restrict__ weights, int W, int E, int top, int scoring) {
+                 int* __restrict__ experts, float* __restrict__ weights, int n_tokens, int W, int E, int top, int scoring, int vec) {
     pdl_trigger();
+    extern __shared__ float mr_smem[];
+    float* zs = mr_smem;                                   // [TOKENS][E]
+    TH* hs = reinterpret_cast<TH*>(zs + (TOKENS * E + 3) / 4 * 4);      // [TOKENS][W]
+    const int t0 = blockIdx.x * TOKENS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int here = min(TOKENS, n_tokens - t0);
     pdl_wait();
     h = pdl_fresh(h);
-    extern __shared__ float mr_smem[];
-    float* hs = mr_smem;             // [W]
-    float* zs = hs + W;              // [E]
-    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    for (int i = tid; i < W; i += 256) hs[i] = to_f32(h[(size_t)t * ldh + i]);
-    __syncthreads();
-    for (int e = warp; e < E; e += 8) {
-        const float* w = wr + (size_t)e * W;
-        float s = 0.0f;
-        for (int i = lane; i < W; i += 32) s = fmaf(w[i], hs[i], s);
-        s = warp_sum(s);
-        if (lane == 0) zs[e] = bias != nullptr ? s + bias[e] : s;
+    constexpr int PIECE = 16 / (int)sizeof(TH);
+    if (W % PIECE == 0 && ldh % PIECE == 0 && ((uintptr_t)h & 15) == 0) {
+        const int per = W / PIECE;
+        for (int i = tid; i < TOKENS * per; i += MR_THREADS) {
+            const int j = i / per, c = (i - j * per) * PIECE;
+            *reinterpret_cast<uint4*>(hs + j * W + c) =
+                j < here ? *reinterpret_cast<const uint4*>(h + (size_t)(t0 + j) * ldh + c) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    } else {
+        for (int j = 0; j < TOKENS; j++)
+            for (int i = tid; i < W; i += MR_THREADS) hs[j * W + i] = j < here ? h[(size_t)(t0 + j) * ldh + i] : from_f32<TH>(0.0f);
     }
     __syncthreads();
-    if (warp == 0) {
+    for (int e = warp; e < E; e += MR_WARPS) {
+        const float* w = wr + (size_t)e * W;
+        float s[TOKENS];
+#pragma unroll
+        for (int j = 0; j < TOKENS; j++) s[j] = 0.0f;
+        if (vec) {
+#pragma unroll (TOKENS == 1 ? 8 : 2)
+            for (int i = lane * 4; i < W; i += 128) {
+                const float4 wv = __ldg(reinterpret_cast<const float4*>(w + i));
+#pragma unroll
+                for (int j = 0; j < TOKENS; j++) {
+                    const float4 x = mr_load4(hs + j * W + i);
+                    s[j] = fmaf(wv.x, x.x, s[j]);
+                    s[j] = fmaf(wv.y, x.y, s[j]);
+                    s[j] = fmaf(wv.z, x.z, s[j]);
+                    s[j] = fmaf(wv.w, x.w, s[j]);
+                }
+            }
+        } else {
+            for (int i = lane; i < W; i += 32) {
+                const float wv = w[i];
+#pragma unroll
+                for (int j = 0; j < TOKENS; j++) s[j] = fmaf(wv, to_f32(hs[j * W + i]), s[j]);
+            }
+        }
+        const float b = bias != nullptr ? bias[e] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < TOKENS; j++) {
+            const float z = warp_sum(s[j]);
+            if (lane == 0) zs[j * E + e] = z + b;
+        }
+    }
+    __syncthreads();
+    if (warp < here) {
         // `top` rounds of: the largest logit not yet taken, lowest index on ties
+        const int t = t0 + warp;
+        float* z = zs + warp * E;
         float zmax = 0.0f, denom = 0.0f;
         for (int k = 0; k < top; k++) {
             float best = -INFINITY;
             int best_e = 0x7fffffff;
             for (int e = lane; e < E; e += 32) {
-                const float v = zs[e];
+                const float v = z[e];
                 if (v > best || (v == best && e < best_e)) { best = v; best_e = e; }
             }
 #pragma unroll
@@ -91,7 +142,7 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
             if (lane == 0) {
                 experts[(size_t)t * top + k] = best_e;
                 weights[(size_t)t * top + k] = p;
-                zs[best_e] = -INFINITY;
+                z[best_e] = -INFINITY;
             }
             __syncwarp();
         }
@@ -100,22 +151,40 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
     }
 }
 
+template <typename TH, int TOKENS>
+static int moe_route_launch(const void* h, long long ldh, const float* wr, const float* bias, int* experts, float* weights, int n_tokens, int W, int E,
+                            int top, int scoring, cudaStream_t s) {
+    const size_t smem = sizeof(float) * ((TOKENS * (size_t)E + 3) / 4 * 4) + sizeof(TH) * TOKENS * (size_t)W;
+    static bool done[HB_MAX_DEVICES] = {};
+    if (smem > 48 * 1024 && !done[hb_device_slot()]) {
+        cudaError_t e = cudaFuncSetAttribute(moe_route_kernel<TH, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return hb_fail("moe_route: %s", cudaGetErrorString(e));
+        done[hb_device_slot()] = true;
+    }
+    const int vec = W % 4 == 0 && ((uintptr_t)wr & 15) == 0 ? 1 : 0;
+    hb_launch(moe_route_kernel<TH, TOKENS>, dim3((n_tokens + TOKENS - 1) / TOKENS), dim3(MR_THREADS), smem, s, (const TH*)h, ldh, wr, bias, experts, weights,
+              n_tokens, W, E, top, scoring, vec);
+    return hb_check_launch("moe_route");
+}
+
 extern "C" int hb_moe_route(const void* h, int h_dtype, long long ldh, const float* w_router, const float* bias, int* experts, float* weights,
                             int n_tokens, int width, int n_experts, int top, int scoring, void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top >= 1 && top <= n_experts, "moe_route: bad sizes");
     HB_REQUIRE(scoring == 0 || scoring == 1, "moe_route: scoring %d (0 softmax over the chosen, 1 sigmoid)", scoring);
-    const size_t smem = sizeof(float) * ((size_t)width + n_experts);
-    HB_REQUIRE(smem <= 48 * 1024, "moe_route: width + experts = %d is too wide", width + n_experts);
+    HB_REQUIRE(h_dtype == HB_BF16 || h_dtype == HB_F32, "moe_route: unsupported dtype %d", h_dtype);
+    const int elem = h_dtype == HB_BF16 ? 2 : 4;
+    const size_t row = (size_t)width * elem + sizeof(float) * (size_t)n_experts + 16;
+    HB_REQUIRE(row <= 200 * 1024, "moe_route: width + experts = %d is too wide", width + n_experts);
+    // tokens to a block: many where the step brings them and shared memory holds their rows
+    const bool eight = n_tokens >= 512 && 8 * row <= 100 * 1024, four = n_tokens >= 64 && 4 * row <= 100 * 1024;
     cudaStream_t s = (cudaStream_t)stream;
-    if (h_dtype == HB_BF16)
-        hb_launch(moe_route_kernel<bf16>, dim3(n_tokens), dim3(256), smem, s, (const bf16*)h, ldh, w_router, bias, experts, weights, width, n_experts, top,
-                  scoring);
-    else if (h_dtype == HB_F32)
-        hb_launch(moe_route_kernel<float>, dim3(n_tokens), dim3(256), smem, s, (const float*)h, ldh, w_router, bias, experts, weights, width, n_experts, top,
-                  scoring);
-    else return hb_fail("moe_route: unsupported dtype %d", h_dtype);
-    return hb_check_launch("moe_route");
+#define HB_MR(TH, N) return moe_route_launch<TH, N>(h, ldh, w_router, bias, experts, weights, n_tokens, width, n_experts, top, scoring, s)
+    if (h_dtype == HB_BF16) { if (eight) HB_MR(bf16, 8); if (four) HB_MR(bf16, 4); HB_MR(bf16, 1); }
+    if (eight) HB_MR(float, 8);
+    if (four) HB_MR(float, 4);
+    HB_MR(float, 1);
+#undef HB_MR
 }
 
 template <typename TH>

@@ -11,6 +11,7 @@ names the size; no op returns a wrong result for an odd size.
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes
 import os
 from typing import Optional
@@ -60,11 +61,11 @@ _SIGNATURES = {
     "hb_gemm_general": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int,
                         _c_int, _c_ptr],
     "hb_gemm_tc": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                   _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr],
+                   _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_int, _c_float, _c_float, _c_ptr],
     "hb_gemm_tc_fold": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                        _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                        _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_int, _c_float, _c_float, _c_ptr, _c_ptr],
     "hb_gemm_tc2": [_c_ptr, _c_ll, _c_ptr, _c_ll, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int,
-                    _c_ptr],
+                    _c_float, _c_float, _c_ptr],
     "hb_attention_general": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
                              _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr],
     "hb_attention_decode": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_int, _c_int,
@@ -332,6 +333,8 @@ class Ops:
         # greedy pick: (maximum, index) of each range of a row, and a counter per row (kept zero)
         self._argmax_scratch = torch.empty(2 * 1024 * self.ARGMAX_MAX_PARTS, dtype=torch.int32, device=self.device)
         self._argmax_counters = torch.zeros(1024, dtype=torch.int32, device=self.device)
+        self._side = None               # the second stream and its split-K scratch (beside)
+        self.use_second_stream = True   # tests switch it off
         self._retired = []              # outgrown scratch, kept alive for graphs that captured it
         self._splits_cache = {}
         self.use_tcgen05_attention = True   # head size 128 prefill on tcgen05 (else the mma.sync kernel)
@@ -367,6 +370,35 @@ class Ops:
             raise KernelError(self.lib.hb_last_error().decode("utf-8", "replace"))
         if self.call_log is not None:
             self.call_log.append(name)
+
+    # ------------------------------------------------------------------ two chains of kernels at once
+    BESIDE_MAX_TOKENS = 64         # steps of more tokens fill the device by themselves
+
+    def can_run_beside(self, tokens: int) -> bool:
+        """Whether a step of so many tokens gains from a second stream (``beside``)."""
+        return bool(self.use_second_stream and 0 < tokens <= self.BESIDE_MAX_TOKENS)
+
+    @contextlib.contextmanager
+    def beside(self):
+        """What is launched inside runs on a second stream, behind everything launched so far and beside what is launched
+        next, until ``join``: for two chains of kernels that share inputs only.  The products inside have split-K scratch of
+        their own.  Works in eager steps and while a graph is captured (the graph then has two branches)."""
+        if self._side is None:
+            self._side = (torch.cuda.Stream(self.device), torch.empty_like(self._splitk_partials), torch.zeros_like(self._splitk_counters))
+        stream, partials, counters = self._side
+        stream.wait_stream(torch.cuda.current_stream(self.device))
+        mine = (self._splitk_partials, self._splitk_counters)
+        self._splitk_partials, self._splitk_counters = partials, counters
+        try:
+            with torch.cuda.stream(stream):
+                yield
+        finally:
+            self._side = (stream, self._splitk_partials, self._splitk_counters)
+            self._splitk_partials, self._splitk_counters = mine
+
+    def join(self) -> None:
+        """What is launched next waits for everything launched inside ``beside``."""
+        torch.cuda.current_stream(self.device).wait_stream(self._side[0])
 
     # ------------------------------------------------------------------ timeline
     def timeline_begin(self, capacity: int = 1 << 16, events: bool = False) -> None:
@@ -868,6 +900,8 @@ class Ops:
     def reset_status(self) -> None:
         self.status.zero_()
         self._splitk_counters.zero_()
+        if self._side is not None:
+            self._side[2].zero_()
         self._decode_counters.zero_()
         self._argmax_counters.zero_()
 
@@ -893,15 +927,16 @@ class Ops:
 
     SCHEDULES = {None: 0, "auto": 0, "tiles": 1, "stream_k": 2, "cut_first": 3}
 
-    def _gemm_tc(self, a, w, out, mode: int, N: int, up_row0: int = 0, schedule=None, fold=None) -> None:
+    def _gemm_tc(self, a, w, out, mode: int, N: int, up_row0: int = 0, schedule=None, fold=None, clamp=None) -> None:
         M, K = a.shape
+        unit = (float(clamp[1]), float(clamp[0])) if clamp is not None else (0.0, 0.0)       # (alpha, limit); alpha 0: silu
         packed = 1 if isinstance(w, PackedWeight) else 0
         ldw = 64 if packed else _rows(w, "linear weight")
         if fold is None and (schedule == "pairs" or (schedule is None and self.use_pair_gemm and self.lib.hb_gemm_tc2_wanted(M, N, K)
                                                      and not (mode == 3 and N % 8))):
             # many tokens: CTA pairs (cta_group::2) on 256 x 256 tiles
             self._call("hb_gemm_tc2", a.data_ptr(), _rows(a, "linear input"), w.data_ptr(), ldw, w.shape[0], out.data_ptr(),
-                       _rows(out, "linear output"), M, N, K, mode, up_row0, self.error_flag.data_ptr(), packed, self._stream())
+                       _rows(out, "linear output"), M, N, K, mode, up_row0, self.error_flag.data_ptr(), packed, *unit, self._stream())
             self.launches += 1
             return
         sched = self.SCHEDULES[schedule]
@@ -916,7 +951,7 @@ class Ops:
         args = (a.data_ptr(), _rows(a, "linear input"), w.data_ptr(), ldw,
                 w.shape[0], out.data_ptr(), _rows(out, "linear output"), M, N, K, mode, up_row0, sched,
                 self._splitk_partials.data_ptr(), self._splitk_partials.numel(), self._splitk_counters.data_ptr(),
-                self._splitk_counters.numel(), self.error_flag.data_ptr(), packed)
+                self._splitk_counters.numel(), self.error_flag.data_ptr(), packed, *unit)
         if fold is None:
             self._call("hb_gemm_tc", *args, self._stream())
         else:
@@ -1001,8 +1036,12 @@ class Ops:
                    1 if accumulate else 0, self._stream())
         self.launches += 1
 
-    def linear_swiglu(self, h, w_gate_up, act, workspace, cap: int, schedule=None, scale: Optional[PreparedNorm] = None) -> None:
-        """``act = silu(h Wg^T) * (h Wu^T)`` with ``w_gate_up = [Wg; Wu]``; ``scale`` as in ``linear``."""
+    def linear_swiglu(self, h, w_gate_up, act, workspace, cap: int, schedule=None, scale: Optional[PreparedNorm] = None,
+                      clamp=None) -> None:
+        """``act = silu(h Wg^T) * (h Wu^T)`` with ``w_gate_up = [Wg; Wu]``; ``scale`` as in ``linear``.  ``clamp = (limit, alpha)``: the
+        clamped unit of ``glu_clamp`` instead (alpha not zero)."""
+        if clamp is not None and float(clamp[1]) == 0.0:
+            raise KernelError("linear_swiglu: the clamped unit needs an alpha that is not zero")
         T = h.shape[0]
         inter = act.shape[1]
         if w_gate_up.shape[0] != 2 * inter or act.shape[0] != T:
@@ -1011,16 +1050,19 @@ class Ops:
                 and _rows(act, "swiglu output") % 8 == 0):
             bands = isinstance(w_gate_up, PackedWeight) and w_gate_up.gate_up_bands
             self._gemm_tc(h, w_gate_up, act, 3, inter, up_row0=-1 if bands else inter, schedule=schedule,
-                          fold=self._scale_fold(scale, T) if scale is not None else None)
+                          fold=self._scale_fold(scale, T) if scale is not None else None, clamp=clamp)
             return
         if scale is not None:
             raise KernelError("linear_swiglu: operands that the tensor-core product refuses cannot take a prepared norm")
         if isinstance(w_gate_up, PackedWeight):
             w_gate_up = w_gate_up.unpacked()
-        gu = workspace.buffer("swiglu.gate_up", (cap, 2 * inter), torch.float32 if act.dtype == torch.float32
+        gu = workspace.buffer("swiglu.gate_up", (cap, 2 * inter), torch.float32 if act.dtype == torch.float32 or clamp is not None
                               else torch.bfloat16)[:T]
         self.linear(h, w_gate_up, gu)
-        self.silu_mul(gu, act)
+        if clamp is not None:
+            self.glu_clamp(gu, act, *clamp)
+        else:
+            self.silu_mul(gu, act)
 
     # ------------------------------------------------------------------ attention
     def decode_splits_for(self, batch: int, kv_heads: int, max_pages: int, head_dim: int = 128) -> int:

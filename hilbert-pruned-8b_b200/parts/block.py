@@ -434,7 +434,8 @@ class ParallelPreNormBlock(Block):
     results in 32-bit buffers of their own; a mixture of experts hands its experts' results on unsummed
     (``FeedForward.weighs_entries``).  One kernel forms the whole sum, adds the vector that the next plan entry adds in front of
     itself (``adds_vector``) and makes the next layer's norm output from the new row, where that layer asks for it
-    (``fold_request`` / ``prepare_next``, the protocol of the sandwich block)."""
+    (``fold_request`` / ``prepare_next``, the protocol of the sandwich block).  In steps of few tokens the two sublayers run
+    on two streams at once (``Ops.beside``)."""
 
     ROLES = {"norm": NORMS, "mixer": MIXERS, "mixer_scale": RESIDUAL_SCALES, "feed_forward": FEED_FORWARDS, "feed_forward_scale": RESIDUAL_SCALES}
     OPTIONAL = ("feed_forward", "feed_forward_scale")
@@ -470,19 +471,28 @@ class ParallelPreNormBlock(Block):
         if prepared is not NORMED:
             self.norm.forward(x, h)
         y = ws.buffer("block.branch", (cap, x.shape[1]), torch.float32)[:T]
-        SandwichBlock._run(self.mixer, y, (h, y, step, cache, state, append))
-        terms = {}
-        if self.ff is not None:
-            if self.fuse_entries and getattr(self.ff, "weighs_entries", False):
-                rows, n, weights, base = self.ff.forward_weighted(h, step)
-                terms = {"entries": rows, "n_sum": n, "entry_weights": weights, "z": base}
-            else:
-                z = ws.buffer("block.second_branch", (cap, x.shape[1]), torch.float32)[:T]
-                SandwichBlock._run(self.ff, z, (h, z, step))
-                terms = {"z": z}
-            terms["b"] = self.ff_scale.factors
+        terms, ops = {}, self.ctx.ops
+        if self.ff is not None and ops.can_run_beside(T):
+            # few tokens: neither sublayer fills the device, so the feed-forward runs on a second stream
+            with ops.beside():
+                terms = self._feed(h, step, x.shape[1])
+            SandwichBlock._run(self.mixer, y, (h, y, step, cache, state, append))
+            ops.join()
+        else:
+            SandwichBlock._run(self.mixer, y, (h, y, step, cache, state, append))
+            if self.ff is not None:
+                terms = self._feed(h, step, x.shape[1])
         ahead = prepare_next if (self.fuse_norms and isinstance(prepare_next, NormAhead) and tuple(prepare_next[3].shape) == tuple(x.shape)) else None
         if ahead is not None:
             terms.update(then=(ahead[0], ahead[2], ahead[1]), then_out=ahead[3])
-        self.ctx.ops.parallel_sum(x, y=y, a=self.mixer_scale.factors, vector=vector, **terms)
+        ops.parallel_sum(x, y=y, a=self.mixer_scale.factors, vector=vector, **terms)
         return NORMED if ahead is not None else None
+
+    def _feed(self, h, step, width: int):
+        """Runs the feed-forward; its result as the terms of ``Ops.parallel_sum``."""
+        if self.fuse_entries and getattr(self.ff, "weighs_entries", False):
+            rows, n, weights, base = self.ff.forward_weighted(h, step)
+            return {"entries": rows, "n_sum": n, "entry_weights": weights, "z": base, "b": self.ff_scale.factors}
+        z = self.ctx.workspace.buffer("block.second_branch", (self.ctx.max_step_tokens, width), torch.float32)[: step.num_tokens]
+        SandwichBlock._run(self.ff, z, (h, z, step))
+        return {"z": z, "b": self.ff_scale.factors}

@@ -15,12 +15,15 @@ from .base import FEED_FORWARDS, FeedForward, ParamSpec
 
 @FEED_FORWARDS.register("swiglu")
 class SwiGLU(FeedForward):
+    NAMES = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
+
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
         self.hidden = int(spec.params["hidden_size"])
         self.inter = int(spec.params["intermediate_size"])
         # the tensors' names below the part's prefix: (gate, up, down)
-        self.names = tuple(spec.get("tensor_names", ("gate_proj.weight", "up_proj.weight", "down_proj.weight")))
+        self.names = tuple(spec.get("tensor_names", self.NAMES))
+        self.clamp = None                     # (limit, alpha) of the clamped unit
         self.w_gate_up = None
         self.w_down = None
 
@@ -49,7 +52,7 @@ class SwiGLU(FeedForward):
         ops, ws, T = self.ctx.ops, self.ctx.workspace, step.num_tokens
         cap = self.ctx.max_step_tokens
         act = ws.buffer("swiglu.act", (cap, self.inter), self.ctx.dtype)[:T]
-        ops.linear_swiglu(h, self.w_gate_up, act, ws, cap, scale=prepared)
+        ops.linear_swiglu(h, self.w_gate_up, act, ws, cap, scale=prepared, clamp=self.clamp)
         return ops.linear(act, self.w_down, residual, accumulate=accumulate, prepare=prepare if accumulate else None)
 
 
@@ -86,29 +89,24 @@ class GatedGelu(FeedForward):
     def weight_bytes(self) -> int:
         return sum(w.numel() * w.element_size() for w in (self.w_gate_up, self.w_down))
 
-    def _unit(self, gate_up, act) -> None:
-        self.ctx.ops.gelu_unit(gate_up, act, "tanh_gated")
-
     def forward(self, h, residual, step, accumulate: bool = True):
         ops, ws, T, cap = self.ctx.ops, self.ctx.workspace, step.num_tokens, self.ctx.max_step_tokens
         first = self.w_gate_up.shape[0]
         gu = ws.buffer(f"gated_gelu.gate_up.{first}", (cap, first), torch.float32)[:T]
         ops.linear(h, self.w_gate_up, gu)
         act = ws.buffer("gated_gelu.act", (cap, self.inter), self.ctx.dtype)[:T]
-        self._unit(gu, act)
+        ops.gelu_unit(gu, act, "tanh_gated")
         ops.linear(act, self.w_down, residual, accumulate=accumulate)
 
 
 @FEED_FORWARDS.register("clamped_glu")
-class ClampedGLU(GatedGelu):
+class ClampedGLU(SwiGLU):
     """``residual += Wd (g sigmoid(alpha g) (u + 1))`` with ``g = min(Wg h, limit)`` and ``u = clamp(Wu h, -limit, limit)``; ``alpha`` is 1.702
-    unless the spec says otherwise.  Gate and up weights are one matrix product with a 32-bit result; the activation reads it
-    unrounded."""
+    unless the spec says otherwise.  The unit reads the products' unrounded 32-bit results, in the product's epilogue where the
+    tensor-core kernel applies."""
+
+    NAMES = ("gate", "up", "down")
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
-        self.limit = float(spec.params["limit"])
-        self.alpha = float(spec.get("alpha", 1.702))
-
-    def _unit(self, gate_up, act) -> None:
-        self.ctx.ops.glu_clamp(gate_up[:, : 2 * self.inter], act, self.limit, self.alpha)
+        self.clamp = (float(spec.params["limit"]), float(spec.get("alpha", 1.702)))
