@@ -227,7 +227,7 @@ int hb_latent_scatter(const void* kv, long long ldkv, const void* k_cache, const
                       const int* seq_pos0, int window, int n_seqs, int max_pages, int n_heads, int d, int dr, int dv, int rank, int hd_out, int vd_out, void* k_out, void* v_out, int n_pages,
                       void* stream);
 int hb_head_linear(const float* in, long long ldi, long long in_head, const void* w, int w_dtype, void* out, int out_dtype, long long ldo,
-                   long long out_head, const float* gate, long long ldg, int n_tokens, int n_heads, int n_in, int n_out, void* stream);
+                   long long out_head, const float* gate, long long ldg, int n_tokens, int n_heads, int n_in, int n_out, int tensor_cores, void* stream);
 // Short causal convolution with bias, activation and state; selective state-space scan (selective_scan.cu)
 int hb_conv_act(const float* x, long long ldx, const float* conv_w, const float* conv_b, int taps, float* state, long long state_stride,
                 const int* state_slots, const int* seq_start, void* out, int out_dtype, long long ldo, int n_seqs, int max_new, int C,
@@ -253,11 +253,11 @@ int hb_moe_glu(const void* h, int h_dtype, long long ldh, const void* w_gate, co
 int hb_moe_down(const void* act, int act_dtype, long long lda, const void* w_down, int w_dtype, const int* offsets, const int* order,
                 const int* tiles, int max_tiles, int top, float* down, long long ldd, int width, int ff, int tensor_cores, void* stream);
 // experts non-null: entries whose expert number is n_real or more are identity experts (their result is the row of h)
-// The two products on tcgen05 over plan tiles of 128 rows (moe_tc.cu): the inputs in the plan's order, then unit 0 (second product) or 1 to 3
+// The two products on tcgen05 over plan tiles of 16 or 128 rows (moe_tc.cu): the inputs in the plan's order, then unit 0 (second product) or 1 to 3
 int hb_moe_gather(const void* h, long long ldh, const int* offsets, int n_experts, const int* order, int top, void* rows, int n_entries, int width,
                   void* stream);
 int hb_moe_tc(const void* a, int n_entries, const void* w0, const void* w1, int n_experts, const int* offsets, const int* order, const int* tiles,
-              int max_tiles, int unit, void* out, long long ldo, int N, int K, float limit, float alpha, const float* in_weights, int sms,
+              int max_tiles, int tile_rows, int unit, void* out, long long ldo, int N, int K, float limit, float alpha, const float* in_weights, int sms,
               int* error_flag, void* stream);
 int hb_moe_combine(const float* down, long long ldd, const float* weights, int top, float* out, long long ldo, int n_tokens, int width,
                    int accumulate, const int* experts, int n_real, const void* h, int h_dtype, long long ldh, void* stream);

@@ -12,10 +12,11 @@
 //    whole pieces of four numbers go through latent_queries, a token's pieces to a block.
 //  * latent_gather, latent_scatter: keys and values of every head written out for steps of many tokens (see there).
 //  * head_linear: out[t, h, :] = W_h in[t, h, :] for every head, W given as [heads][n_in][n_out]
-//    (the output index contiguous), 32-bit accumulation on the FP32 pipe; optionally times
-//    sigmoid(gate[t, h]).  Serves both q' (W = Wuk as stored) and the values (W = Wuv transposed).
+//    (the output index contiguous), 32-bit accumulation on the tensor cores (bfloat16 weights, the
+//    inputs as two bfloat16 terms) or on the FP32 pipe; optionally times sigmoid(gate[t, h]).  Serves both q' (W = Wuk as stored) and the values (W = Wuv transposed).
 #include "api.h"
 #include "common.cuh"
+#include "mma.cuh"
 
 #define LP_THREADS 128
 
@@ -396,12 +397,116 @@ head_linear_kernel(const float* __restrict__ in, long long ldi, long long in_hea
     }
 }
 
+// The same on the tensor cores (mma.sync m16n8k16) for bfloat16 weights: a block owns 16 tokens x HM_COLS columns of one head, brings
+// all of its weights [n_in][HM_COLS] and the tokens' inputs in at once, and its warps share the input features out (their partial
+// sums are added in a fixed order).  The 32-bit inputs enter as TWO bfloat16 terms, hi = bf16(x) and lo = bf16(x - hi), i.e. exact
+// to 16 mantissa bits.
+#define HM_THREADS 128
+#define HM_COLS 32
+#define HM_WST (HM_COLS + 8)         // bfloat16 per staged weight row
+
+static size_t hm_smem(int n_in) {
+    const int k16 = (n_in + 15) / 16 * 16;
+    return (size_t)k16 * HM_WST * 2 + 2 * (size_t)16 * (k16 + 8) * 2 + (size_t)4 * 16 * HM_COLS * 4;
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(HM_THREADS)
+head_linear_mma_kernel(const float* __restrict__ in, long long ldi, long long in_head, const bf16* __restrict__ w, TO* __restrict__ out, long long ldo,
+                       long long out_head, const float* __restrict__ gate, long long ldg, int n_tokens, int n_in, int n_out) {
+    pdl_trigger();
+    extern __shared__ __align__(128) unsigned char hm_mem[];
+    const int k16 = (n_in + 15) / 16 * 16, xst = k16 + 8;
+    bf16* Ws = reinterpret_cast<bf16*>(hm_mem);                    // [k16][HM_WST]
+    bf16* Xh = Ws + (size_t)k16 * HM_WST;                          // [16][xst]
+    bf16* Xl = Xh + 16 * xst;
+    float* part = reinterpret_cast<float*>(Xl + 16 * xst);         // [4 warps][16][HM_COLS]
+    const int t0 = blockIdx.x * 16, h = blockIdx.y, n0 = blockIdx.z * HM_COLS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int cols = min(HM_COLS, n_out - n0);                     // (a multiple of 8)
+    const bf16* wh = w + (size_t)h * n_in * n_out + n0;
+    const uint32_t ws_addr = (uint32_t)__cvta_generic_to_shared(Ws);
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    // the weights do not depend on the kernel in front
+    for (int i = tid; i < k16 * (HM_COLS / 8); i += HM_THREADS) {
+        const int k = i / (HM_COLS / 8), c = (i % (HM_COLS / 8)) * 8;
+        if (k < n_in && c < cols) cp_async_16(ws_addr + (uint32_t)(k * HM_WST + c) * 2, wh + (size_t)k * n_out + c);
+        else *reinterpret_cast<uint4*>(Ws + k * HM_WST + c) = zero;
+    }
+    cp_async_commit();
+    pdl_wait();
+    in = pdl_fresh(in);
+    gate = pdl_fresh(gate);
+    for (int i = tid; i < 16 * k16; i += HM_THREADS) {
+        const int j = i / k16, k = i - j * k16;
+        const float x = (t0 + j < n_tokens && k < n_in) ? in[(size_t)(t0 + j) * ldi + (size_t)h * in_head + k] : 0.0f;
+        const bf16 hi = __float2bfloat16_rn(x);
+        Xh[j * xst + k] = hi;
+        Xl[j * xst + k] = __float2bfloat16_rn(x - __bfloat162float(hi));
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[HM_COLS / 8][4];
+#pragma unroll
+    for (int i = 0; i < HM_COLS / 8; i++) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
+    const uint32_t xh_addr = (uint32_t)__cvta_generic_to_shared(Xh), xl_addr = (uint32_t)__cvta_generic_to_shared(Xl);
+    const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8, b_row = ((lane >> 3) & 1) * 8 + (lane & 7), b_chunk = lane >> 4;
+#pragma unroll 4
+    for (int ks = warp; ks < k16 / 16; ks += 4) {
+        uint32_t ah[4], al[4];
+        const uint32_t off = (uint32_t)(a_row * xst + ks * 16 + a_col) * 2;
+        ldmatrix_x4(ah, xh_addr + off);
+        ldmatrix_x4(al, xl_addr + off);
+#pragma unroll
+        for (int p = 0; p < HM_COLS / 16; p++) {
+            uint32_t bf[4];
+            ldmatrix_x4_trans(bf, ws_addr + (uint32_t)((ks * 16 + b_row) * HM_WST + p * 16 + b_chunk * 8) * 2);
+            mma_bf16_16816(acc[2 * p], ah, bf[0], bf[1]);
+            mma_bf16_16816(acc[2 * p], al, bf[0], bf[1]);
+            mma_bf16_16816(acc[2 * p + 1], ah, bf[2], bf[3]);
+            mma_bf16_16816(acc[2 * p + 1], al, bf[2], bf[3]);
+        }
+    }
+    const int r0 = lane >> 2, c0 = (lane & 3) * 2;
+#pragma unroll
+    for (int i = 0; i < HM_COLS / 8; i++) {
+        *reinterpret_cast<float2*>(part + (warp * 16 + r0) * HM_COLS + i * 8 + c0) = make_float2(acc[i][0], acc[i][1]);
+        *reinterpret_cast<float2*>(part + (warp * 16 + r0 + 8) * HM_COLS + i * 8 + c0) = make_float2(acc[i][2], acc[i][3]);
+    }
+    __syncthreads();
+    for (int i = tid; i < 16 * HM_COLS; i += HM_THREADS) {
+        const int j = i / HM_COLS, c = i % HM_COLS, t = t0 + j;
+        if (t >= n_tokens || c >= cols) continue;
+        float v = (part[i] + part[16 * HM_COLS + i]) + (part[2 * 16 * HM_COLS + i] + part[3 * 16 * HM_COLS + i]);
+        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
+        out[(size_t)t * ldo + (size_t)h * out_head + n0 + c] = from_f32<TO>(v);
+    }
+}
+
+template <typename TO>
+static int head_linear_mma(const float* in, long long ldi, long long in_head, const void* w, void* out, long long ldo, long long out_head,
+                           const float* gate, long long ldg, int n_tokens, int n_heads, int n_in, int n_out, cudaStream_t s) {
+    static bool done[HB_MAX_DEVICES] = {};
+    if (!done[hb_device_slot()]) {
+        cudaError_t e = cudaFuncSetAttribute(head_linear_mma_kernel<TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return hb_fail("head_linear: %s", cudaGetErrorString(e));
+        done[hb_device_slot()] = true;
+    }
+    hb_launch(head_linear_mma_kernel<TO>, dim3((n_tokens + 15) / 16, n_heads, (n_out + HM_COLS - 1) / HM_COLS), dim3(HM_THREADS), hm_smem(n_in), s, in, ldi, in_head,
+              (const bf16*)w, (TO*)out, ldo, out_head, gate, ldg, n_tokens, n_in, n_out);
+    return hb_check_launch("head_linear");
+}
+
 extern "C" int hb_head_linear(const float* in, long long ldi, long long in_head, const void* w, int w_dtype, void* out, int out_dtype,
                               long long ldo, long long out_head, const float* gate, long long ldg, int n_tokens, int n_heads, int n_in,
-                              int n_out, void* stream) {
+                              int n_out, int tensor_cores, void* stream) {
     if (n_tokens == 0) return 0;
     HB_REQUIRE(n_tokens > 0 && n_heads > 0 && n_heads <= 65535 && n_in > 0 && n_out > 0, "head_linear: bad sizes");
     HB_REQUIRE((n_out + 31) / 32 <= 65535, "head_linear: too many output columns");
+    if (tensor_cores && w_dtype == HB_BF16 && n_out % 8 == 0 && ((uintptr_t)w & 15) == 0 && hm_smem(n_in) <= 200 * 1024 && n_out <= 65535 * HM_COLS) {
+        cudaStream_t ms = (cudaStream_t)stream;
+        if (out_dtype == HB_BF16) return head_linear_mma<bf16>(in, ldi, in_head, w, out, ldo, out_head, gate, ldg, n_tokens, n_heads, n_in, n_out, ms);
+        if (out_dtype == HB_F32) return head_linear_mma<float>(in, ldi, in_head, w, out, ldo, out_head, gate, ldg, n_tokens, n_heads, n_in, n_out, ms);
+    }
     // narrow tiles where wide ones would not fill the SMs once (a matter of the product's sizes only)
     const int cols = ((long long)n_heads * ((n_out + 63) / 64) < 148) ? 32 : 64;
     dim3 grid((n_tokens + HL_TOKENS - 1) / HL_TOKENS, n_heads, (n_out + cols - 1) / cols);

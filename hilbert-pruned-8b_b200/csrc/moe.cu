@@ -69,6 +69,9 @@ moe_route_kernel(const TH* __restrict__ h, long long ldh, const float* __restric
     TH* hs = reinterpret_cast<TH*>(zs + (TOKENS * E + 3) / 4 * 4);      // [TOKENS][W]
     const int t0 = blockIdx.x * TOKENS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int here = min(TOKENS, n_tokens - t0);
+    if (TOKENS == 1)                                       // no kernel of a step writes the matrix: ask for it while the one in front runs
+        for (int e = warp; e < E; e += MR_WARPS)
+            for (int i = lane * 32; i < W; i += 32 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(wr + (size_t)e * W + i));
     pdl_wait();
     h = pdl_fresh(h);
     constexpr int PIECE = 16 / (int)sizeof(TH);
@@ -346,7 +349,8 @@ extern "C" int hb_moe_tile_rows(int tensor_cores) { return tensor_cores ? MM_BM 
 extern "C" int hb_moe_plan(const int* experts, int n_entries, int n_experts, int tile_rows, int* offsets, int* order, int* tiles, void* stream) {
     if (n_entries == 0) return 0;
     HB_REQUIRE(n_entries > 0 && n_experts > 0 && n_experts <= 4096, "moe_plan: bad sizes");
-    HB_REQUIRE(tile_rows == MOE_BM || tile_rows == MM_BM || tile_rows == 128, "moe_plan: tiles of %d rows (%d, %d or 128 are built)", tile_rows, MOE_BM, MM_BM);
+    HB_REQUIRE(tile_rows == MOE_BM || tile_rows == MM_BM || tile_rows == 16 || tile_rows == 128,
+               "moe_plan: tiles of %d rows (16, %d, %d or 128 are built)", tile_rows, MOE_BM, MM_BM);
     hb_launch(moe_plan_kernel, dim3(1), dim3(1024), sizeof(int) * 2 * n_experts, (cudaStream_t)stream, experts, n_entries, n_experts, tile_rows,
               offsets, order, tiles);
     return hb_check_launch("moe_plan");

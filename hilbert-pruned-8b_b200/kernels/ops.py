@@ -107,7 +107,7 @@ _SIGNATURES = {
     "hb_latent_scatter": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                           _c_ptr, _c_ptr, _c_int, _c_ptr],
     "hb_head_linear": [_c_ptr, _c_ll, _c_ll, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ll, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_int,
-                       _c_ptr],
+                       _c_int, _c_ptr],
     "hb_conv_act": [_c_ptr, _c_ll, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int,
                     _c_int, _c_ptr],
     "hb_selective_scan": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ll, _c_ptr,
@@ -119,7 +119,7 @@ _SIGNATURES = {
     "hb_moe_down": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int,
                     _c_ptr],
     "hb_moe_gather": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr],
-    "hb_moe_tc": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_float, _c_float,
+    "hb_moe_tc": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_float, _c_float,
                   _c_ptr, _c_int, _c_ptr, _c_ptr],
     "hb_moe_combine": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ptr],
     "hb_moe_route_scores": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
@@ -1583,7 +1583,8 @@ class Ops:
             raise KernelError("head_linear: rows are too short for the heads")
         gp, ldg = self._head_gate(gate, T, heads)
         self._call("hb_head_linear", x.data_ptr(), _rows(x, "head_linear input"), int(in_head), w.data_ptr(), _code(w), out.data_ptr(),
-                   _code(out), _rows(out, "head_linear output"), int(out_head), gp, ldg, T, heads, n_in, n_out, self._stream())
+                   _code(out), _rows(out, "head_linear output"), int(out_head), gp, ldg, T, heads, n_in, n_out,
+                   1 if self.use_tensor_cores else 0, self._stream())
         self.launches += 1
 
     # ------------------------------------------------------------------ selective state-space scan
@@ -1745,15 +1746,15 @@ class Ops:
     def moe_max_tiles(self, entries: int, n_experts: int, tile_rows: int) -> int:
         return int(self.lib.hb_moe_max_tiles(int(entries), int(n_experts), int(tile_rows)))
 
-    MOE_TC_ROWS = 24                # steps with so many entries per expert (on average) run the experts' products on tcgen05
+    MOE_TC_ROWS = 8                 # steps with so many entries per expert (on average) cut them into tiles of 128 rows, others of 16
 
     def moe_experts(self, h, experts, weights, w_gate, w_up, w_down, limit: float, alpha: float, out, accumulate: bool, workspace,
                     cap: int, tag: str = "", identity: bool = False, unit: str = "clamped_glu", weigh: str = "output"):
         """``out (+)= sum_k weights[t, k] * expert_{experts[t, k]}(h[t])`` with the experts' weights stacked ``[experts, ff,
         width]`` (gate, up) and ``[experts, width, ff]`` (down) in the activations' dtype and the clamped gated unit of
         ``glu_clamp`` between them.  Four or five launches: plan, (gathered inputs,) gate/up with activation, down, weighted sum.
-        bfloat16 operands whose rows are multiples of 8 elements run the products on the tensor cores (``use_tensor_cores``; tcgen05 for
-        ``MOE_TC_ROWS`` entries per expert or more, else mma.sync), all others on the FP32 pipe.
+        bfloat16 operands whose rows are multiples of 8 elements run the products on the tensor cores (``use_tensor_cores``; tcgen05, or
+        mma.sync without ``use_tcgen05_experts``), all others on the FP32 pipe.
         ``w_up`` None: experts of one matrix, ``act = gelu_erf(w_gate h)`` (``limit`` and ``alpha`` unused).  ``identity``: expert
         numbers from the stack's size on are identity experts, whose result is ``h[t]`` itself.  ``unit`` "silu_glu": ``silu(gate) * up``
         between the products.  ``weigh`` "input": an expert is fed ``weights[t, k] * h[t]`` and its result is added as it is.
@@ -1775,11 +1776,11 @@ class Ops:
         most = cap * top
         tc = 1 if (self.use_tensor_cores and h.dtype == torch.bfloat16 and W % 8 == 0 and F % 8 == 0 and _rows(h, "expert input") % 8 == 0
                    and h.data_ptr() % 16 == 0) else 0
-        # many rows per expert: tcgen05 over tiles of 128 rows; fewer: mma.sync over tiles of 64 (or the FP32 pipe over tiles of 32)
-        umma = bool(tc and self.use_tcgen05_experts and entries >= self.MOE_TC_ROWS * E)
-        tile_rows = 128 if umma else int(self.lib.hb_moe_tile_rows(tc))
+        # tensor cores: tcgen05 over tiles of 128 rows, or of 16 where experts have few; else the FP32 pipe over tiles of 32
+        umma = bool(tc and self.use_tcgen05_experts)
+        tile_rows = (128 if entries >= self.MOE_TC_ROWS * E else 16) if umma else int(self.lib.hb_moe_tile_rows(tc))
         max_tiles = self.moe_max_tiles(entries, E, tile_rows)
-        plan = workspace.buffer("moe.plan" + tag, (E + 1 + most + 1 + 2 * self.moe_max_tiles(most, E, 32),), torch.int32)
+        plan = workspace.buffer("moe.plan" + tag, (E + 1 + most + 1 + 2 * self.moe_max_tiles(most, E, 16),), torch.int32)
         offsets, order, tiles = plan[: E + 1], plan[E + 1: E + 1 + most], plan[E + 1 + most:]
         act = workspace.buffer("moe.act" + tag, (most, F), h.dtype)
         down = workspace.buffer("moe.down" + tag, (most, W), torch.float32)
@@ -1791,10 +1792,10 @@ class Ops:
             rows = workspace.buffer("moe.rows" + tag, (most, W), h.dtype)
             self._call("hb_moe_gather", h.data_ptr(), _rows(h, "expert input"), offsets.data_ptr(), E, order.data_ptr(), top, rows.data_ptr(), entries, W, s)
             self._call("hb_moe_tc", rows.data_ptr(), entries, w_gate.data_ptr(), w_up.data_ptr() if w_up is not None else None, E, offsets.data_ptr(),
-                       order.data_ptr(), tiles.data_ptr(), max_tiles, unit_code, act.data_ptr(), F, F, W, float(limit), float(alpha), in_weights,
+                       order.data_ptr(), tiles.data_ptr(), max_tiles, tile_rows, unit_code, act.data_ptr(), F, F, W, float(limit), float(alpha), in_weights,
                        self.sm_count, self.error_flag.data_ptr(), s)
             self._call("hb_moe_tc", act.data_ptr(), entries, w_down.data_ptr(), None, E, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles,
-                       0, down.data_ptr(), W, W, F, 0.0, 0.0, None, self.sm_count, self.error_flag.data_ptr(), s)
+                       tile_rows, 0, down.data_ptr(), W, W, F, 0.0, 0.0, None, self.sm_count, self.error_flag.data_ptr(), s)
             self.launches += 4
         else:
             self._call("hb_moe_glu", h.data_ptr(), _code(h), _rows(h, "expert input"), w_gate.data_ptr(),
