@@ -256,7 +256,7 @@ int hb_moe_down(const void* act, int act_dtype, long long lda, const void* w_dow
 // The two products on tcgen05 over plan tiles of 16 or 128 rows (moe_tc.cu): the inputs in the plan's order, then unit 0 (second product) or 1 to 3
 int hb_moe_gather(const void* h, long long ldh, const int* offsets, int n_experts, const int* order, int top, void* rows, int n_entries, int width,
                   void* stream);
-int hb_moe_tc(const void* a, int n_entries, const void* w0, const void* w1, int n_experts, const int* offsets, const int* order, const int* tiles,
+int hb_moe_tc(const void* a, int n_entries, const void* w, int n_experts, const int* offsets, const int* order, const int* tiles,
               int max_tiles, int tile_rows, int unit, void* out, long long ldo, int N, int K, float limit, float alpha, const float* in_weights, int sms,
               int* error_flag, void* stream);
 int hb_moe_combine(const float* down, long long ldd, const float* weights, int top, float* out, long long ldo, int n_tokens, int width,

@@ -16,8 +16,9 @@
 #define AG_THREADS 256
 #define AG_WARPS 8
 #define AG_KEYS HB_PAGE_TOKENS
-#define AG_SST (AG_KEYS + 4)           // floats per row of scores
-#define AG_PST (AG_KEYS + 8)           // bfloat16 per row of weights
+// A row of scores (AG_KEYS floats) becomes a row of weights in its place: AG_KEYS leading terms, then AG_KEYS rests, bfloat16
+#define AG_SST (AG_KEYS + 4)           // floats per row
+#define AG_PST (2 * AG_SST)            // the same in bfloat16
 #define AG_LOG2E 1.4426950408889634f
 #define AG_SMEM_MAX (220 * 1024)
 #define AG_MAX_SPLITS 64
@@ -35,7 +36,7 @@ static bool ag_sizes(int group, int hd, int vd, int v_in_k, AgSizes& z, int& mt)
     z.vst = v_in_k ? z.kst : z.vd16 + 8;
     z.stage_elems = (size_t)AG_KEYS * (z.kst + (v_in_k ? 0 : z.vst));
     const size_t rows = 16 * (size_t)mt;
-    const size_t fixed = rows * z.kst * 2 + rows * AG_SST * 4 + 2 * rows * AG_PST * 2 + 2 * rows * 4;
+    const size_t fixed = rows * z.kst * 2 + rows * AG_SST * 4 + 2 * rows * 4;
     const size_t stage = z.stage_elems * 2;
     if (fixed + 2 * stage > AG_SMEM_MAX) return false;
     // two blocks on an SM where that leaves two stages, up to four stages
@@ -61,9 +62,9 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
     bf16* stage0 = reinterpret_cast<bf16*>(ag_smem);
     bf16* Qs = stage0 + (size_t)stages * stage_elems;           // [ROWS][kst]
     float* Ss = reinterpret_cast<float*>(Qs + ROWS * kst);      // [ROWS][AG_SST]
-    bf16* Ph = reinterpret_cast<bf16*>(Ss + ROWS * AG_SST);     // [ROWS][AG_PST]
-    bf16* Pl = Ph + ROWS * AG_PST;
-    float* c_s = reinterpret_cast<float*>(Pl + ROWS * AG_PST);  // [ROWS]: the accumulators' factor of this page
+    bf16* Ph = reinterpret_cast<bf16*>(Ss);                     // [ROWS][AG_PST]: leading terms, and AG_KEYS further on the rests
+    bf16* Pl = Ph + AG_KEYS;
+    float* c_s = Ss + ROWS * AG_SST;                            // [ROWS]: the accumulators' factor of this page
     float* l_s = c_s + ROWS;                                    // [ROWS]: the rows' sums, at the end
 
     const int split = blockIdx.x, splits = gridDim.x, t = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -76,14 +77,12 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
     const int pg0 = lo / AG_KEYS, pg1 = p / AG_KEYS + 1, per = (pg1 - pg0 + splits - 1) / splits;
     const int p_begin = pg0 + split * per, n_it = max(0, min(pg1, p_begin + per) - p_begin);
 
-    // what stays zero: the keys' and queries' columns behind the head (their products must vanish) and the weights of rows
-    // that no head owns
+    // what stays zero: the keys' and queries' columns behind the head (their products must vanish)
     if (hd16 > hd)
         for (int i = tid; i < stages * AG_KEYS; i += AG_THREADS) {
             bf16* row = stage0 + (size_t)(i / AG_KEYS) * stage_elems + (size_t)(i % AG_KEYS) * kst;
             for (int d = hd; d < hd16; d++) row[d] = __float2bfloat16_rn(0.0f);
         }
-    for (int i = tid; i < ROWS * AG_PST; i += AG_THREADS) Ph[i] = Pl[i] = __float2bfloat16_rn(0.0f);
     if (tid < ROWS) c_s[tid] = 1.0f;
 
     pdl_wait();
@@ -149,7 +148,7 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
         l_r[i] = with_sink && lane == 0 ? 1.0f : 0.0f;
     }
     const uint32_t q_base = (uint32_t)__cvta_generic_to_shared(Qs), ph_base = (uint32_t)__cvta_generic_to_shared(Ph);
-    const uint32_t pl_base = (uint32_t)__cvta_generic_to_shared(Pl);
+    const uint32_t pl_base = ph_base + AG_KEYS * 2;
     const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8, r0 = lane >> 2;
     const int v_row = ((lane >> 3) & 1) * 8 + (lane & 7), v_chunk = lane >> 4;
 
@@ -197,7 +196,12 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
 #pragma unroll
         for (int i = 0; i < 2 * MT; i++) {
             const int row = warp + 8 * i;
-            if (row >= rows) continue;                              // the same for the whole warp
+            if (row >= rows) {                                      // (the same for the whole warp) no head owns this row: no weights
+                const uint32_t none = 0u;
+                *reinterpret_cast<uint32_t*>(Ph + row * AG_PST + 2 * lane) = none;
+                *reinterpret_cast<uint32_t*>(Pl + row * AG_PST + 2 * lane) = none;
+                continue;
+            }
             const float s0 = (key0 >= lo && key0 <= p) ? Ss[row * AG_SST + lane] * scale_log2e : -INFINITY;
             const float s1 = (key1 >= lo && key1 <= p) ? Ss[row * AG_SST + lane + 32] * scale_log2e : -INFINITY;
             const float m_new = fmaxf(m_r[i], warp_max(fmaxf(s0, s1)));
@@ -206,6 +210,7 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
             m_r[i] = m_new;
             l_r[i] = l_r[i] * corr + p0 + p1;
             const bf16 hi0 = __float2bfloat16_rn(p0), hi1 = __float2bfloat16_rn(p1);
+            __syncwarp();                                           // every lane has its scores: the weights may take their place
             Ph[row * AG_PST + lane] = hi0;
             Ph[row * AG_PST + lane + 32] = hi1;
             Pl[row * AG_PST + lane] = __float2bfloat16_rn(p0 - __bfloat162float(hi0));

@@ -3,14 +3,18 @@
 // stream of weights): plan tiles of 16 rows, units of 64 weight rows, so that the units share the weights out evenly over
 // the SMs, and sixteen stages in flight; the MMA still works on 128 rows, of which the others are whatever lies behind the tile.
 //
+// The experts' weights are packed in bands of 64 rows: [expert][band][K block][64 rows][64 columns], zeros beyond a matrix, so that a CTA
+// that walks along K reads one sequential range of memory, 8 KB per K block and band.  A band of a gated unit's two matrices
+// holds 32 gate rows and the 32 up rows of the same features.
+//
 // moe_gather:  rows[slot] = h[token of the entry at that slot]: the experts' inputs in the plan's order, so that the rows of an
 //              expert's tile are neighbours and TMA can copy them.  (The rows of a tile behind an expert's last one belong to
 //              the next expert; their results are not stored.)
 // moe_tc:      one persistent CTA per SM walks units (plan tile, column block).  Accumulators: 128 rows (lanes of tensor memory) x BR
 //              columns (the unit's weight rows), two buffers, so that the epilogue of a unit runs while the next one is computed.
-//              Gated units (two matrices): the first half of the columns are gate features, the second half the up values of
+//              Gated units (two matrices): of every 64 columns the first 32 are gate features, the others the up values of
 //              the same features, and the epilogue is the activation; else BR columns of the one matrix.
-//   warp 0     TMA producer: per K block of 64 the tile's rows and twice BR / 2 weight rows
+//   warp 0     TMA producer: per K block of 64 the tile's rows and BR / 64 bands of weights
 //   warp 1     owns tensor memory; one thread issues the MMAs (128 x BR x 16)
 //   warps 2-5  epilogue, one thread per row
 // First product (MODE 1, 2, 3 as in moe_act.cuh): act[slot], bfloat16; with in_weights both products' results are multiplied by
@@ -58,9 +62,9 @@ __device__ __forceinline__ bool mt_wait(uint32_t bar, uint32_t parity, volatile 
 
 template <int MODE, typename TO, int ROWS, int BR>
 __global__ void __launch_bounds__(TC_THREADS, 1)
-moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b0, const __grid_constant__ CUtensorMap map_b1,
+moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
               const int* __restrict__ offsets, const int* __restrict__ order, const int* __restrict__ tiles, TO* __restrict__ out, long long ldo,
-              int N, int K, int n_blocks, float limit, float alpha, const float* __restrict__ in_weights, int* __restrict__ error_flag) {
+              int N, int K, int n_blocks, int bands, float limit, float alpha, const float* __restrict__ in_weights, int* __restrict__ error_flag) {
     constexpr bool GLU = MODE == 1 || MODE == 3;
     using S = mt_shape<ROWS, BR>;
     constexpr int STAGES = S::STAGES;
@@ -108,9 +112,8 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
             int g = 0;
             bool alive = true;
             for (int u = blockIdx.x; u < units && alive; u += gridDim.x) {
-                const int ti = u / n_blocks, n0 = (u - ti * n_blocks) * COLS;
-                const int e = tiles[1 + 2 * ti], r0 = tiles[2 + 2 * ti];
-                const int w_row = e * N + n0;
+                const int ti = u / n_blocks, e = tiles[1 + 2 * ti], r0 = tiles[2 + 2 * ti];
+                const int band0 = (u - ti * n_blocks) * (BR / 64);                   // the unit's first band of the expert's
                 for (int kb = 0; kb < kb_total; kb++, g++) {
                     const int s = g % STAGES;
                     if (!mt_wait(empty0 + 8 * s, ((g / STAGES) & 1) ^ 1, abort_flag)) {
@@ -121,9 +124,12 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
                     }
                     const uint32_t b = b_smem + s * S::B_BYTES, bar = full0 + 8 * s;
                     mbar_expect_tx(bar, S::A_BYTES + S::B_BYTES);
-                    tma_load_2d(b, &map_b0, bar, kb * TC_BK, w_row);
-                    if (GLU) tma_load_2d(b + S::B_BYTES / 2, &map_b1, bar, kb * TC_BK, w_row);
-                    else tma_load_2d(b + S::B_BYTES / 2, &map_b0, bar, kb * TC_BK, w_row + BR / 2);
+#pragma unroll
+                    for (int j = 0; j < BR / 64; j++) {
+                        // (a unit may reach beyond the expert's last band: its results there are not stored)
+                        const int band = min(band0 + j, bands - 1);
+                        tma_load_2d(b + j * 64 * TC_BK * 2, &map_b, bar, 0, ((e * bands + band) * kb_total + kb) * 64);
+                    }
                     tma_load_2d(a_smem + s * S::A_BYTES, &map_a, bar, kb * TC_BK, r0);
                 }
             }
@@ -188,8 +194,9 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
             for (int c = 0; c < COLS; c += 16) {
                 if (n0 + c >= N) break;                              // (the same for all)
                 float v0[16], v1[16];
-                tmem_ld16(lane_addr + c, v0);
-                if (GLU) tmem_ld16(lane_addr + BR / 2 + c, v1);
+                const int at = GLU ? (c >> 5) * 64 + (c & 31) : c;
+                tmem_ld16(lane_addr + at, v0);
+                if (GLU) tmem_ld16(lane_addr + at + 32, v1);
                 if (here) {
 #pragma unroll
                     for (int j = 0; j < 16; j++) v0[j] = moe_first_act<MODE>(v0[j] * rw, GLU ? v1[j] * rw : 0.0f, limit, alpha);
@@ -227,7 +234,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
 }
 
 template <int MODE, typename TO, int ROWS, int BR>
-static int moe_tc_launch(const void* a, int n_entries, const void* w0, const void* w1, int n_experts, const int* offsets, const int* order,
+static int moe_tc_launch(const void* a, int n_entries, const void* w, int n_experts, const int* offsets, const int* order,
                          const int* tiles, int max_tiles, void* out, long long ldo, int N, int K, float limit, float alpha, const float* in_weights,
                          int sms, int* error_flag, cudaStream_t s) {
     constexpr int SMEM = mt_shape<ROWS, BR>::SMEM;
@@ -237,16 +244,18 @@ static int moe_tc_launch(const void* a, int n_entries, const void* w0, const voi
         if (e != cudaSuccess) return hb_fail("moe_tc: cannot reserve %d bytes of shared memory: %s", SMEM, cudaGetErrorString(e));
         done[hb_device_slot()] = true;
     }
-    CUtensorMap ma, m0, m1;
+    const int per_band = MODE == 1 || MODE == 3 ? 32 : 64, bands = (N + per_band - 1) / per_band, kbs = (K + TC_BK - 1) / TC_BK;
+    const long long rows = (long long)n_experts * bands * kbs * 64;
+    HB_REQUIRE(rows < (1ll << 31), "moe_tc: too many weight rows");
+    CUtensorMap ma, mb;
     if (tc_make_map(&ma, a, n_entries, K, K, ROWS)) return 1;
-    if (tc_make_map(&m0, w0, (long long)n_experts * N, K, K, BR / 2)) return 1;
-    if (tc_make_map(&m1, w1 != nullptr ? w1 : w0, (long long)n_experts * N, K, K, BR / 2)) return 1;
+    if (tc_make_map(&mb, w, rows, TC_BK, TC_BK, 64)) return 1;
     constexpr int COLS = MODE == 1 || MODE == 3 ? BR / 2 : BR;
     const int n_blocks = (N + COLS - 1) / COLS;
     const long long most = (long long)max_tiles * n_blocks;
     const int grid = (int)(most < sms ? most : sms);
-    cudaError_t e = hb_launch(moe_tc_kernel<MODE, TO, ROWS, BR>, dim3(grid), dim3(TC_THREADS), SMEM, s, ma, m0, m1, offsets, order, tiles, (TO*)out, ldo, N, K,
-                              n_blocks, limit, alpha, in_weights, error_flag);
+    cudaError_t e = hb_launch(moe_tc_kernel<MODE, TO, ROWS, BR>, dim3(grid), dim3(TC_THREADS), SMEM, s, ma, mb, offsets, order, tiles, (TO*)out, ldo, N, K,
+                              n_blocks, bands, limit, alpha, in_weights, error_flag);
     if (e != cudaSuccess) return hb_fail("moe_tc: launch failed: %s", cudaGetErrorString(e));
     return hb_check_launch("moe_tc");
 }
@@ -261,23 +270,23 @@ extern "C" int hb_moe_gather(const void* h, long long ldh, const int* offsets, i
     return hb_check_launch("moe_gather");
 }
 
-// a: bfloat16 [n_entries][K] in the plan's order (tiles of tile_rows rows, 16 or 128); w0, w1: bfloat16 stacks [n_experts][N][K] (w1 null: one matrix).  unit 0: out
-// float32 [n_entries][N] at the entries' rows; 1: clamped gated unit, 2: exact gelu of w0, 3: silu-gated unit: out bfloat16 at the slots' rows.
-extern "C" int hb_moe_tc(const void* a, int n_entries, const void* w0, const void* w1, int n_experts, const int* offsets, const int* order,
+// a: bfloat16 [n_entries][K] in the plan's order (tiles of tile_rows rows, 16 or 128); w: the packed
+// bands of the experts' [N][K] (unit 1 and 3: of both matrices).  unit 0: out float32 [n_entries][N] at the entries' rows; 1: clamped gated
+// unit, 2: exact gelu of the one matrix, 3: silu-gated unit: out bfloat16 at the slots' rows.
+extern "C" int hb_moe_tc(const void* a, int n_entries, const void* w, int n_experts, const int* offsets, const int* order,
                          const int* tiles, int max_tiles, int tile_rows, int unit, void* out, long long ldo, int N, int K, float limit, float alpha,
                          const float* in_weights, int sms, int* error_flag, void* stream) {
     if (n_entries == 0) return 0;
     HB_REQUIRE(n_entries > 0 && n_experts > 0 && max_tiles > 0 && N > 0 && K > 0 && N % 8 == 0 && K % 8 == 0 && ldo >= N && ldo % 8 == 0 && sms > 0,
                "moe_tc: bad sizes (rows of a multiple of 8 elements expected)");
-    HB_REQUIRE((long long)n_experts * N < (1ll << 31), "moe_tc: too many weight rows");
-    HB_REQUIRE(unit >= 0 && unit <= 3 && (w1 != nullptr) == (unit == 1 || unit == 3), "moe_tc: unit %d (1 and 3: two matrices, 0 and 2: one)", unit);
-    HB_REQUIRE((((uintptr_t)a | (uintptr_t)w0 | (uintptr_t)w1 | (uintptr_t)out) & 15) == 0 && error_flag != nullptr, "moe_tc: operands must be 16-byte aligned");
+    HB_REQUIRE(unit >= 0 && unit <= 3, "moe_tc: unit %d (0 to 3)", unit);
+    HB_REQUIRE((((uintptr_t)a | (uintptr_t)w | (uintptr_t)out) & 15) == 0 && error_flag != nullptr, "moe_tc: operands must be 16-byte aligned");
     HB_REQUIRE(tile_rows == 16 || tile_rows == 128, "moe_tc: plan tiles of %d rows (16 or 128 are built)", tile_rows);
     cudaStream_t s = (cudaStream_t)stream;
 #define HB_MT(U, TO)                                                                                                                       \
-    return tile_rows == 16 ? moe_tc_launch<U, TO, 16, 64>(a, n_entries, w0, w1, n_experts, offsets, order, tiles, max_tiles, out, ldo, N, K, limit,  \
+    return tile_rows == 16 ? moe_tc_launch<U, TO, 16, 64>(a, n_entries, w, n_experts, offsets, order, tiles, max_tiles, out, ldo, N, K, limit,  \
                                                           alpha, in_weights, sms, error_flag, s)                                             \
-                           : moe_tc_launch<U, TO, 128, 256>(a, n_entries, w0, w1, n_experts, offsets, order, tiles, max_tiles, out, ldo, N, K,       \
+                           : moe_tc_launch<U, TO, 128, 256>(a, n_entries, w, n_experts, offsets, order, tiles, max_tiles, out, ldo, N, K,       \
                                                             limit, alpha, in_weights, sms, error_flag, s)
     if (unit == 0) HB_MT(0, float);
     if (unit == 1) HB_MT(1, bf16);

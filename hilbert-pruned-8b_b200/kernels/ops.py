@@ -119,7 +119,7 @@ _SIGNATURES = {
     "hb_moe_down": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int,
                     _c_ptr],
     "hb_moe_gather": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr],
-    "hb_moe_tc": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_float, _c_float,
+    "hb_moe_tc": [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_float, _c_float,
                   _c_ptr, _c_int, _c_ptr, _c_ptr],
     "hb_moe_combine": [_c_ptr, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ptr],
     "hb_moe_route_scores": [_c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
@@ -293,6 +293,48 @@ class PackedWeight:
         return self.data.data_ptr()
 
 
+class PackedExperts:
+    """The bfloat16 matrices ``[experts, rows, cols]`` of one product of a mixture's experts, or with ``paired`` the gate and the up
+    matrices of their first product, stored for the tensor-core kernel (``moe_tc``) in bands of 64 rows: ``data`` is ``[experts, bands,
+    column blocks, 64, 64]``, zero beyond ``rows`` and ``cols``, so that a CTA that walks along the columns of a band reads one
+    sequential range of memory.  A paired band holds 32 gate rows and the 32 up rows of the same features."""
+
+    def __init__(self, data: torch.Tensor, rows: int, cols: int, paired: bool):
+        self.data, self.rows, self.cols, self.paired = data, int(rows), int(cols), bool(paired)
+
+    @classmethod
+    def pack(cls, w: torch.Tensor, up: Optional[torch.Tensor] = None) -> "PackedExperts":
+        E, rows, cols = w.shape
+        per = 64 if up is None else 32
+        bands, blocks = -(-rows // per), -(-cols // 64)
+        data = torch.zeros(E, bands, blocks, 64, 64, dtype=w.dtype, device=w.device)
+        for e in range(E):                     # expert by expert: no second copy of the whole stack
+            for at, m in ((0, w[e]),) if up is None else ((0, w[e]), (32, up[e])):
+                full = torch.zeros(bands * per, blocks * 64, dtype=w.dtype, device=w.device)
+                full[:rows, :cols] = m
+                data[e, :, :, at: at + per] = full.view(bands, per, blocks, 64).transpose(1, 2)
+        return cls(data, rows, cols, up is not None)
+
+    def unpacked(self):
+        """The matrices ``[experts, rows, cols]`` again: ``(w, None)``, or with ``paired`` ``(gate, up)``."""
+        E, bands, blocks = self.data.shape[:3]
+        def out(at, per):
+            m = self.data[:, :, :, at: at + per].transpose(2, 3).reshape(E, bands * per, blocks * 64)
+            return m[:, : self.rows, : self.cols].contiguous()
+        return (out(0, 32), out(32, 32)) if self.paired else (out(0, 64), None)
+
+    @property
+    def shape(self):
+        return (self.data.shape[0], self.rows, self.cols)
+
+    @property
+    def dtype(self):
+        return self.data.dtype
+
+    def element_size(self) -> int:
+        return self.data.element_size()
+
+
 class Ops:
     """The kernels bound to one device."""
 
@@ -344,7 +386,7 @@ class Ops:
         self.use_mma_attention = True
         self.use_flash_sink_attention = True    # steps of many tokens: attention_sink_prefill where it is built
         self.use_tcgen05_sink_attention = True  # and on tcgen05 (attention_sink_prefill_tc) where heads are not mixed
-        self.use_tcgen05_experts = True         # experts' products of many rows on tcgen05 (moe_tc); tests compare both
+        self.use_tcgen05_experts = True         # experts' weights are packed for tcgen05 (moe_tc) when they are bound; tests compare both
         self.use_group_attention = True         # steps of few tokens whose heads are not mixed: attention_group where it is built
         self.use_mma_pool_attention = True      # steps of many tokens: attention_pool_prefill where it is built (tests compare both)
         # Decode attention that rotates the new queries and key and appends to the cache itself
@@ -1748,25 +1790,40 @@ class Ops:
 
     MOE_TC_ROWS = 8                 # steps with so many entries per expert (on average) cut them into tiles of 128 rows, others of 16
 
+    def pack_experts(self, w_gate, w_up, w_down):
+        """``(first, second)`` as PackedExperts where the tensor-core kernel takes these stacks (bfloat16 on this device, rows of a
+        multiple of 8 elements; ``w_up`` None: one matrix in front of the activation), else None."""
+        if not (self.use_tcgen05_experts and self.use_tensor_cores and w_gate.dtype == w_down.dtype == torch.bfloat16
+                and w_gate.device == self.device and w_gate.shape[1] % 8 == 0 and w_gate.shape[2] % 8 == 0):
+            return None
+        return PackedExperts.pack(w_gate, w_up), PackedExperts.pack(w_down)
+
     def moe_experts(self, h, experts, weights, w_gate, w_up, w_down, limit: float, alpha: float, out, accumulate: bool, workspace,
                     cap: int, tag: str = "", identity: bool = False, unit: str = "clamped_glu", weigh: str = "output"):
         """``out (+)= sum_k weights[t, k] * expert_{experts[t, k]}(h[t])`` with the experts' weights stacked ``[experts, ff,
         width]`` (gate, up) and ``[experts, width, ff]`` (down) in the activations' dtype and the clamped gated unit of
         ``glu_clamp`` between them.  Four or five launches: plan, (gathered inputs,) gate/up with activation, down, weighted sum.
-        bfloat16 operands whose rows are multiples of 8 elements run the products on the tensor cores (``use_tensor_cores``; tcgen05, or
-        mma.sync without ``use_tcgen05_experts``), all others on the FP32 pipe.
-        ``w_up`` None: experts of one matrix, ``act = gelu_erf(w_gate h)`` (``limit`` and ``alpha`` unused).  ``identity``: expert
+        Stacked bfloat16 operands whose rows are multiples of 8 elements run on the tensor cores too (``use_tensor_cores``; mma.sync), all
+        others on the FP32 pipe.
+        Packed experts (``pack_experts``) run on tcgen05.  ``w_up`` None (``unit`` "gelu"): experts of one matrix, ``act = gelu_erf(w_gate h)`` (``limit`` and ``alpha`` unused).  ``identity``: expert
         numbers from the stack's size on are identity experts, whose result is ``h[t]`` itself.  ``unit`` "silu_glu": ``silu(gate) * up``
         between the products.  ``weigh`` "input": an expert is fed ``weights[t, k] * h[t]`` and its result is added as it is.
         ``out`` None: no sum; returns the experts' results, float32 ``[tokens * top, width]`` (engine scratch), for a caller whose
         own kernel adds a token's rows (with their weights unless ``weigh`` is "input")."""
-        self._dev(h, experts, weights, w_gate, w_up, w_down, out)
+        self._dev(h, experts, weights, *((w.data if isinstance(w, PackedExperts) else w) for w in (w_gate, w_up, w_down)), out)
+        if w_up is None and not isinstance(w_gate, PackedExperts):
+            unit = "gelu"
         if (out is None and identity) or weigh not in ("input", "output") or (weigh == "input" and identity):
             raise KernelError("moe_experts: identity experts have their results weighted and summed here")
         T, W = h.shape
         E, F = w_gate.shape[0], w_gate.shape[1]
         top = experts.shape[1]
-        if tuple(w_gate.shape) != (E, F, W) or (w_up is not None and tuple(w_up.shape) != (E, F, W)) or tuple(w_down.shape) != (E, W, F) \
+        packed = isinstance(w_gate, PackedExperts)
+        if packed:
+            if not isinstance(w_down, PackedExperts) or w_up is not None or tuple(w_gate.shape) != (E, F, W) or tuple(w_down.shape) != (E, W, F) \
+                    or w_down.paired or w_gate.paired == (unit == "gelu") or h.dtype != torch.bfloat16 or w_gate.dtype != h.dtype or w_down.dtype != h.dtype:
+                raise KernelError("moe_experts: packed experts of both products in the activations' dtype expected")
+        elif tuple(w_gate.shape) != (E, F, W) or (w_up is not None and tuple(w_up.shape) != (E, F, W)) or tuple(w_down.shape) != (E, W, F) \
                 or not (w_gate.is_contiguous() and (w_up is None or w_up.is_contiguous()) and w_down.is_contiguous()) \
                 or not (w_gate.dtype == w_down.dtype == h.dtype) or (w_up is not None and w_up.dtype != h.dtype):
             raise KernelError("moe_experts: stacked contiguous expert weights in the activations' dtype expected")
@@ -1776,8 +1833,10 @@ class Ops:
         most = cap * top
         tc = 1 if (self.use_tensor_cores and h.dtype == torch.bfloat16 and W % 8 == 0 and F % 8 == 0 and _rows(h, "expert input") % 8 == 0
                    and h.data_ptr() % 16 == 0) else 0
-        # tensor cores: tcgen05 over tiles of 128 rows, or of 16 where experts have few; else the FP32 pipe over tiles of 32
-        umma = bool(tc and self.use_tcgen05_experts)
+        # packed experts: tcgen05 over tiles of 128 rows, or of 16 where experts have few
+        umma = bool(tc and packed)
+        if packed and not umma:                # not a product path: only rows the tensor-core kernel refuses get here
+            (w_gate, w_up), (w_down, _) = w_gate.unpacked(), w_down.unpacked()
         tile_rows = (128 if entries >= self.MOE_TC_ROWS * E else 16) if umma else int(self.lib.hb_moe_tile_rows(tc))
         max_tiles = self.moe_max_tiles(entries, E, tile_rows)
         plan = workspace.buffer("moe.plan" + tag, (E + 1 + most + 1 + 2 * self.moe_max_tiles(most, E, 16),), torch.int32)
@@ -1786,15 +1845,15 @@ class Ops:
         down = workspace.buffer("moe.down" + tag, (most, W), torch.float32)
         s = self._stream()
         self._call("hb_moe_plan", experts.data_ptr(), entries, E, tile_rows, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), s)
-        unit_code = 2 if w_up is None else {"clamped_glu": 1, "silu_glu": 3}[unit]
+        unit_code = {"gelu": 2, "clamped_glu": 1, "silu_glu": 3}[unit]
         in_weights = weights.data_ptr() if weigh == "input" else None
         if umma:
             rows = workspace.buffer("moe.rows" + tag, (most, W), h.dtype)
             self._call("hb_moe_gather", h.data_ptr(), _rows(h, "expert input"), offsets.data_ptr(), E, order.data_ptr(), top, rows.data_ptr(), entries, W, s)
-            self._call("hb_moe_tc", rows.data_ptr(), entries, w_gate.data_ptr(), w_up.data_ptr() if w_up is not None else None, E, offsets.data_ptr(),
+            self._call("hb_moe_tc", rows.data_ptr(), entries, w_gate.data.data_ptr(), E, offsets.data_ptr(),
                        order.data_ptr(), tiles.data_ptr(), max_tiles, tile_rows, unit_code, act.data_ptr(), F, F, W, float(limit), float(alpha), in_weights,
                        self.sm_count, self.error_flag.data_ptr(), s)
-            self._call("hb_moe_tc", act.data_ptr(), entries, w_down.data_ptr(), None, E, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles,
+            self._call("hb_moe_tc", act.data_ptr(), entries, w_down.data.data_ptr(), E, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), max_tiles,
                        tile_rows, 0, down.data_ptr(), W, W, F, 0.0, 0.0, None, self.sm_count, self.error_flag.data_ptr(), s)
             self.launches += 4
         else:

@@ -20,7 +20,7 @@ logits as in the plain form, weighted by their sigmoids, not divided by anything
 ``router.b``), which counts for the choice and for the weights; for the routers "top_logits" and "sigmoid".
 
 Tensors below the part's prefix: ``router``, ``e<i>.gate|up|down``, ``shared.gate|up|down``.  The
-experts' matrices are stacked at load time; the routed products gather their rows on the device
+experts' matrices are stacked at load time (and packed for the tensor cores where those take them); the routed products gather their rows on the device
 from a plan that a kernel makes, so a step reads nothing back and decode steps can be captured.
 """
 from __future__ import annotations
@@ -77,6 +77,7 @@ class MixtureOfExperts(FeedForward):
         # or with their weights and the shared expert's result beside them
         self.weighs_entries = not self.identity
         self.b_router = None
+        self.first = None                     # both products' weights packed for the tensor cores (then w_gate and w_up are not kept)
         self.correction = None
         self.gate_col = None
         self.w_router = self.w_gate = self.w_up = self.w_down = self.ws_gate_up = self.ws_down = None
@@ -107,6 +108,10 @@ class MixtureOfExperts(FeedForward):
         self.w_gate = torch.stack([t[f"e{e}.gate"] for e in range(E)]).contiguous() if glu else None
         self.w_up = torch.stack([t[f"e{e}.up"] for e in range(E)]).contiguous()
         self.w_down = torch.stack([t[f"e{e}.down"] for e in range(E)]).contiguous()
+        packed = self.ctx.ops.pack_experts(self.w_gate if glu else self.w_up, self.w_up if glu else None, self.w_down)
+        if packed is not None:
+            self.first, self.w_down = packed
+            self.w_gate = self.w_up = None
         if self.router == "scores":
             self.correction = t["correction"].reshape(-1).to(torch.float32).contiguous()
         if self.shared_ff:
@@ -125,7 +130,7 @@ class MixtureOfExperts(FeedForward):
 
     def weight_bytes(self) -> int:
         # what a decode step of one token reads: the router, `top` experts, the shared expert
-        per = (3 if self.w_gate is not None else 2) * self.ff * self.hidden * self.w_up.element_size()
+        per = (3 if self.glu else 2) * self.ff * self.hidden * self.w_down.element_size()
         shared = sum(w.numel() * w.element_size() for w in (self.ws_gate_up, self.ws_down)) if self.shared_ff else 0
         return self.w_router.numel() * 4 + self.top * per + shared
 
@@ -151,11 +156,11 @@ class MixtureOfExperts(FeedForward):
             ops.moe_route(h, self.w_router, self.top, experts, weights, scoring="sigmoid" if self.router == "sigmoid" else "softmax_chosen",
                           bias=self.b_router)
         if self.unit == "gelu":
-            rows = ops.moe_experts(h, experts, weights, self.w_up, None, self.w_down, 0.0, 0.0, residual, accumulate, ws, cap,
-                                   tag=".gelu", identity=self.identity > 0, weigh=self.weigh)
+            rows = ops.moe_experts(h, experts, weights, self.first if self.first is not None else self.w_up, None, self.w_down, 0.0, 0.0, residual,
+                                   accumulate, ws, cap, tag=".gelu", identity=self.identity > 0, unit="gelu", weigh=self.weigh)
         else:
-            rows = ops.moe_experts(h, experts, weights, self.w_gate, self.w_up, self.w_down, self.limit, self.alpha, residual, accumulate, ws, cap,
-                                   unit=self.unit, weigh=self.weigh)
+            rows = ops.moe_experts(h, experts, weights, self.first if self.first is not None else self.w_gate, self.w_up, self.w_down, self.limit,
+                                   self.alpha, residual, accumulate, ws, cap, unit=self.unit, weigh=self.weigh)
         return rows, weights
 
     def forward(self, h, residual, step, accumulate: bool = True):
