@@ -91,6 +91,23 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
     v_cache = pdl_fresh(v_cache);
     gate = pdl_fresh(gate);
     const int kc = hd / 8, vc = vd / 8;
+    // a thread's 16-byte pieces of a page are AG_THREADS apart: the row and the piece of the row advance by fixed steps
+    const int k_row0 = tid / kc, k_col0 = tid - k_row0 * kc, k_rows_on = AG_THREADS / kc, k_cols_on = AG_THREADS - k_rows_on * kc;
+    const int v_row0 = tid / vc, v_col0 = tid - v_row0 * vc, v_rows_on = AG_THREADS / vc, v_cols_on = AG_THREADS - v_rows_on * vc;
+    auto copy_rows = [&](uint32_t dst, const bf16* src, int per, int st, int r, int c, int rows_on, int cols_on) {
+        const bf16* from = src + (size_t)tid * 8;
+#pragma unroll 2
+        while (r < AG_KEYS) {
+            cp_async_16(dst + (uint32_t)(r * st + c * 8) * 2, from);
+            from += AG_THREADS * 8;
+            r += rows_on;
+            c += cols_on;
+            if (c >= per) {
+                c -= per;
+                r++;
+            }
+        }
+    };
     bool bad_page = false;
     auto load_page = [&](int it) {
         if (it < n_it) {
@@ -103,18 +120,10 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
             bf16* ks = stage0 + (size_t)(it % stages) * stage_elems;
             const bf16* ksrc = k_cache + ((size_t)page * nkv + g) * AG_KEYS * hd;
             const uint32_t kdst = (uint32_t)__cvta_generic_to_shared(ks);
-            for (int i = tid; i < AG_KEYS * kc; i += AG_THREADS) {
-                const int r = i / kc, c = i - r * kc;
-                cp_async_16(kdst + (uint32_t)(r * kst + c * 8) * 2, ksrc + (size_t)i * 8);
-            }
-            if (!v_in_k) {
-                const bf16* vsrc = v_cache + ((size_t)page * nkv + g) * AG_KEYS * vd;
-                const uint32_t vdst = kdst + (uint32_t)(AG_KEYS * kst) * 2;
-                for (int i = tid; i < AG_KEYS * vc; i += AG_THREADS) {
-                    const int r = i / vc, c = i - r * vc;
-                    cp_async_16(vdst + (uint32_t)(r * vst + c * 8) * 2, vsrc + (size_t)i * 8);
-                }
-            }
+            copy_rows(kdst, ksrc, kc, kst, k_row0, k_col0, k_rows_on, k_cols_on);
+            if (!v_in_k)
+                copy_rows(kdst + (uint32_t)(AG_KEYS * kst) * 2, v_cache + ((size_t)page * nkv + g) * AG_KEYS * vd, vc, vst, v_row0, v_col0, v_rows_on,
+                          v_cols_on);
         }
         cp_async_commit();
     };
@@ -231,7 +240,8 @@ attention_group_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __
                     acc[a][b][c][3] *= c1;
                 }
         }
-#pragma unroll
+        // (small code: a block runs few pages, and what it has not yet run comes from L2)
+#pragma unroll 1
         for (int ks = 0; ks < AG_KEYS / 16; ks++) {
             uint32_t ah[MT][4], al[MT][4];
 #pragma unroll

@@ -89,7 +89,7 @@ template <int MODE>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(T2_THREADS, 1)
 gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                 const __grid_constant__ CUtensorMap map_o, const TcParams p, const int tma_out) {
-    constexpr bool SWIGLU = MODE == TC_SWIGLU_BF16;
+    constexpr bool SWIGLU = tc_gated(MODE);
     constexpr int STAGES = T2_STAGES;
     constexpr int STAGE_BYTES = T2_STAGE_BYTES;
     constexpr int TOKENS = T2_TOKENS;
@@ -292,7 +292,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
 #pragma unroll
                         for (int j = 0; j < 16; j++) {
                             const float other = theirs[j * 64 + f];
-                            const float y = gate_thread ? tc_unit(p, v[0][j], other) : tc_unit(p, other, v[1][j]);
+                            const float y = gate_thread ? tc_unit<MODE>(p, v[0][j], other) : tc_unit<MODE>(p, other, v[1][j]);
                             yb[((gate_thread ? 0 : 16) + j) * 64 + f] = __float2bfloat16_rn(y);
                         }
                         fence_async_shared();
@@ -517,6 +517,8 @@ extern "C" int hb_gemm_tc2(const void* a, long long lda, const void* w, long lon
         case TC_STORE_BF16: return launch_tc2<TC_STORE_BF16>(mw, ma, mo, prm, tma_out, pairs, s);
         case TC_STORE_F32: return launch_tc2<TC_STORE_F32>(mw, ma, mo, prm, tma_out, pairs, s);
         case TC_ADD_F32: return launch_tc2<TC_ADD_F32>(mw, ma, mo, prm, tma_out, pairs, s);
-        default: return launch_tc2<TC_SWIGLU_BF16>(mw, ma, mo, prm, tma_out, pairs, s);
+        default:
+            return prm.unit_alpha != 0.0f ? launch_tc2<TC_CLAMPED_BF16>(mw, ma, mo, prm, tma_out, pairs, s)
+                                          : launch_tc2<TC_SWIGLU_BF16>(mw, ma, mo, prm, tma_out, pairs, s);
     }
 }

@@ -7,7 +7,7 @@
 
 template <int BN, int MODE>
 struct TcLayout {
-    static constexpr bool SWIGLU = MODE == TC_SWIGLU_BF16;
+    static constexpr bool SWIGLU = tc_gated(MODE);
     static constexpr int FEAT = SWIGLU ? 64 : TC_BM;                   // output features per tile
     static constexpr int W_BYTES = TC_BM * TC_BK * 2;                  // 16 KB: 128 weight rows
     static constexpr int A_BYTES = BN * TC_BK * 2;
@@ -528,7 +528,7 @@ struct TcLaunch {
 // step of 8 layers at batch 8: 1305 us; with the partial tiles over 11 stages and the second
 // cluster barrier that needs: 1327 us).  32 and 64 tokens: the stages of the plain kernels.
 template <int BN, int MODE, bool FOLD = false>
-using TcClusterLaunch = TcLaunch<BN, MODE, BN == 16 ? (MODE == TC_SWIGLU_BF16 ? 7 : 8) : BN == 32 ? 10 : 8, true, FOLD>;
+using TcClusterLaunch = TcLaunch<BN, MODE, BN == 16 ? (tc_gated(MODE) ? 7 : 8) : BN == 32 ? 10 : 8, true, FOLD>;
 
 template <int BN, int MODE>
 static bool clusters_fit(int size, long long tiles) {
@@ -562,7 +562,9 @@ static int tc_launch_bn_fold(bool cluster, int mode, const CUtensorMap& mw, cons
                 case TC_STORE_BF16: return TcClusterLaunch<BN, TC_STORE_BF16, FOLD>::launch(mw, ma, prm, grid, s);
                 case TC_STORE_F32: return TcClusterLaunch<BN, TC_STORE_F32, FOLD>::launch(mw, ma, prm, grid, s);
                 case TC_ADD_F32: return TcClusterLaunch<BN, TC_ADD_F32, FOLD>::launch(mw, ma, prm, grid, s);
-                default: return TcClusterLaunch<BN, TC_SWIGLU_BF16, FOLD>::launch(mw, ma, prm, grid, s);
+                default:
+                    return prm.unit_alpha != 0.0f ? TcClusterLaunch<BN, TC_CLAMPED_BF16, FOLD>::launch(mw, ma, prm, grid, s)
+                                                  : TcClusterLaunch<BN, TC_SWIGLU_BF16, FOLD>::launch(mw, ma, prm, grid, s);
             }
         } else {
             return hb_fail("gemm_tc: no cluster variant for token tile %d", BN);
@@ -572,7 +574,9 @@ static int tc_launch_bn_fold(bool cluster, int mode, const CUtensorMap& mw, cons
         case TC_STORE_BF16: return TcLaunch<BN, TC_STORE_BF16, STAGES, false, FOLD>::launch(mw, ma, prm, grid, s);
         case TC_STORE_F32: return TcLaunch<BN, TC_STORE_F32, STAGES, false, FOLD>::launch(mw, ma, prm, grid, s);
         case TC_ADD_F32: return TcLaunch<BN, TC_ADD_F32, STAGES, false, FOLD>::launch(mw, ma, prm, grid, s);
-        default: return TcLaunch<BN, TC_SWIGLU_BF16, STAGES, false, FOLD>::launch(mw, ma, prm, grid, s);
+        default:
+            return prm.unit_alpha != 0.0f ? TcLaunch<BN, TC_CLAMPED_BF16, STAGES, false, FOLD>::launch(mw, ma, prm, grid, s)
+                                          : TcLaunch<BN, TC_SWIGLU_BF16, STAGES, false, FOLD>::launch(mw, ma, prm, grid, s);
     }
 }
 

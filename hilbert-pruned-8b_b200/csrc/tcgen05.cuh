@@ -11,7 +11,9 @@
 #define TC_THREADS 192
 #define TC_WAIT_LIMIT (1u << 24)
 
-enum { TC_STORE_BF16 = 0, TC_STORE_F32 = 1, TC_ADD_F32 = 2, TC_SWIGLU_BF16 = 3 };
+enum { TC_STORE_BF16 = 0, TC_STORE_F32 = 1, TC_ADD_F32 = 2, TC_SWIGLU_BF16 = 3, TC_CLAMPED_BF16 = 4 };
+// the epilogues that pair a gate and an up product (the host names both 3; the clamped unit is chosen by TcParams::unit_alpha)
+__host__ __device__ constexpr bool tc_gated(int mode) { return mode == TC_SWIGLU_BF16 || mode == TC_CLAMPED_BF16; }
 
 // ------------------------------------------------------------------------------- PTX
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -207,13 +209,14 @@ struct TcParams {
     const float* scale_sumsq;   // consumer: nullptr: none
     int scale_parts;      // slots per token to add
     float scale_inv_size, scale_eps;
-    // SWIGLU: the unit of a gate and an up value.  unit_alpha 0: silu(g) * u; else the clamped unit g' sigmoid(alpha g') (u' + 1)
-    // with g' = min(g, unit_limit), u' = u clamped to +-unit_limit
+    // the gated epilogues: unit_alpha 0: silu(g) * u; else (TC_CLAMPED_BF16) the clamped unit g' sigmoid(unit_alpha g') (u' + 1) with
+    // g' = min(g, unit_limit), u' = u clamped to +-unit_limit
     float unit_alpha, unit_limit;
 };
 
+template <int MODE>
 __device__ __forceinline__ float tc_unit(const TcParams& p, float g, float u) {
-    if (p.unit_alpha == 0.0f) return silu_fast(g) * u;
+    if (MODE != TC_CLAMPED_BF16) return silu_fast(g) * u;
     g = fminf(g, p.unit_limit);
     u = fminf(fmaxf(u, -p.unit_limit), p.unit_limit);
     return g * (1.0f / (1.0f + expf(-p.unit_alpha * g))) * (u + 1.0f);
@@ -287,7 +290,7 @@ __device__ __forceinline__ void tc_emit_chunk(const TcParams& p, int m0, int n0,
     const bool scaled = FOLD && MODE != TC_ADD_F32 && p.scale_sumsq != nullptr;
 #pragma unroll
     for (int j = 0; j < 16; j++) v[j] = (FOLD && scaled) ? v_in[j] * srow[min(m0 + c + j, p.M - 1)] : v_in[j];
-    if (MODE == TC_SWIGLU_BF16) {
+    if (tc_gated(MODE)) {
         // rows 0..63 of the tile are gate rows, rows 64..127 the up rows of the same
         // features: pair them through shared memory, then store 16 bytes per thread
         float* xf = (float*)xchg + ((c >> 4) & 1) * (16 * 64);
@@ -299,7 +302,7 @@ __device__ __forceinline__ void tc_emit_chunk(const TcParams& p, int m0, int n0,
         asm volatile("bar.sync 1, 128;" ::: "memory");
         if (q < 2) {
 #pragma unroll
-            for (int j = 0; j < 16; j++) yb[j * 64 + row] = __float2bfloat16_rn(tc_unit(p, v[j], xf[j * 64 + row]));
+            for (int j = 0; j < 16; j++) yb[j * 64 + row] = __float2bfloat16_rn(tc_unit<MODE>(p, v[j], xf[j * 64 + row]));
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");
         const int r = et >> 3, ch = et & 7;                 // token row of the chunk, 8-feature group
@@ -438,7 +441,7 @@ __device__ __forceinline__ void tc_emit_flat(const TcParams& p, int m0, int n0, 
         const float sc = scaled ? srow[m] : 1.0f;
         const float v[4] = {FOLD ? acc[i].x * sc : acc[i].x, FOLD ? acc[i].y * sc : acc[i].y, FOLD ? acc[i].z * sc : acc[i].z,
                             FOLD ? acc[i].w * sc : acc[i].w};
-        if (MODE == TC_SWIGLU_BF16) {
+        if (tc_gated(MODE)) {
             // lanes 0..15 hold gate rows 4 * lane .. + 3, lanes 16..31 the up rows of the same features
             float u[4];
 #pragma unroll
@@ -447,7 +450,7 @@ __device__ __forceinline__ void tc_emit_flat(const TcParams& p, int m0, int n0, 
             if (lane < 16 && n < p.N) {
                 bf16 y[4];
 #pragma unroll
-                for (int e = 0; e < 4; e++) y[e] = __float2bfloat16_rn(tc_unit(p, v[e], u[e]));
+                for (int e = 0; e < 4; e++) y[e] = __float2bfloat16_rn(tc_unit<MODE>(p, v[e], u[e]));
                 bf16* o = (bf16*)p.out + (size_t)m * p.ldc + n;
                 if (n + 4 <= p.N) {
                     *reinterpret_cast<uint2*>(o) = *reinterpret_cast<const uint2*>(y);
