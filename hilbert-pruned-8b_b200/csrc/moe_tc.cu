@@ -178,7 +178,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
             const int buf = item & 1;
             const int ti = u / n_blocks, n0 = (u - ti * n_blocks) * COLS;
             const int e = tiles[1 + 2 * ti], r0 = tiles[2 + 2 * ti];
-            const bool here = r0 + row < offsets[e + 1];
+            const bool here = row < ROWS && r0 + row < offsets[e + 1];     // a row of this tile and of this expert
             const int entry = here ? order[r0 + row] : 0;
             const float rw = (MODE != 0 && in_weights != nullptr && here) ? in_weights[entry] : 1.0f;
             TO* dst = out + (size_t)(MODE != 0 ? r0 + row : entry) * ldo + n0;

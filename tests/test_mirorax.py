@@ -252,7 +252,8 @@ def test_biased_router_with_silu_experts_and_a_shared_expert(dtype):
     from hilbert_pruned_8b_b200.parts import FEED_FORWARDS
     g, rnd = torch.Generator().manual_seed(3), _rnd(dtype)
     for n, (width, E, top, ff, shared, T) in enumerate(((24, 3, 2, 10, 7, 1), (64, 6, 2, 32, 64, 5), (64, 5, 1, 24, 0, 333), (40, 1, 1, 8, 8, 70),
-                                                        (128, 40, 6, 64, 192, 90), (56, 4, 4, 40, 20, 33), (264, 4, 2, 200, 64, 700))):
+                                                        (128, 40, 6, 64, 192, 90), (56, 4, 4, 40, 20, 33), (264, 4, 2, 200, 64, 700),
+                                                        (72, 8, 2, 40, 24, 31), (64, 16, 4, 72, 64, 31))):       # (small tiles, and experts with more rows than one holds)
         for tc in ("tcgen05", "mma.sync", None):          # the products' three kernels (where the step has rows enough and bfloat16 for them)
             c = _context(dtype, cap=1024)
             c.ops.use_tensor_cores, c.ops.use_tcgen05_experts = tc is not None, tc == "tcgen05"
@@ -263,6 +264,9 @@ def test_biased_router_with_silu_experts_and_a_shared_expert(dtype):
                  for p in part.params()}
             part.bind({k: (v.to(dtype) if v.dim() == 2 else v).to(DEV) for k, v in w.items()})
             h = (torch.randn(T, width, generator=g) * 1.5).to(torch.bfloat16)
+            if T == 31:
+                w["router.b"][:2] += 12.0                  # every token's choice: 31 rows for an expert
+                part.bind({k: (v.to(dtype) if v.dim() == 2 else v).to(DEV) for k, v in w.items()})
             cfg = {"router": {"experts": E, "top": top}, "shared": {"ff": shared} if shared else None}
             want = moe_ff(h.double(), _double(w), cfg, rnd)
             if top < E and T > 1:                          # the bias does decide
