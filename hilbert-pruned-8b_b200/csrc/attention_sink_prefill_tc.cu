@@ -313,6 +313,33 @@ attn_sink_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_before();
             mbar_arrive(p_full0 + 8 * s);
         }
+        // the row's gates, while the last product runs: 1 / (1 + exp(-g)) of this thread's output columns
+        const int t = t_begin + row_base + r;
+        const float* gr = gate != nullptr && valid ? gate + (size_t)t * ldg : nullptr;
+        const bool each = gr != nullptr && gate_per > 1;
+        float gv[OC];
+#pragma unroll
+        for (int c = 0; c < OC; c++) gv[c] = 1.0f;
+        if (each) {
+            const float* ge = gr + (size_t)head * vd + hf * OC;
+            if (((uintptr_t)ge & 15) == 0) {
+#pragma unroll
+                for (int c = 0; c < OC; c += 4)
+                    if (hf * OC + c < vd) {                    // (vd is a multiple of 8)
+                        const float4 g4 = *reinterpret_cast<const float4*>(ge + c);
+                        gv[c] = g4.x;
+                        gv[c + 1] = g4.y;
+                        gv[c + 2] = g4.z;
+                        gv[c + 3] = g4.w;
+                    }
+            } else {
+#pragma unroll
+                for (int c = 0; c < OC; c++)
+                    if (hf * OC + c < vd) gv[c] = ge[c];
+            }
+#pragma unroll
+            for (int c = 0; c < OC; c++) gv[c] = 1.0f / (1.0f + expf(-gv[c]));
+        }
         if (ok && !mbar_wait(pv_done, (n_it - 1) & 1)) {
             atomicExch(error_flag, 29);
             *abort_flag = 1;
@@ -324,13 +351,10 @@ attn_sink_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (!*abort_flag) {
             tc_fence_after();
             const float lt = xrow[r] + xrow[128 + r];
-            const int t = t_begin + row_base + r;
-            const float* gr = gate != nullptr && valid ? gate + (size_t)t * ldg : nullptr;
             float inv = lt > 0.0f ? 1.0f / lt : 0.0f;
             if (gr != nullptr && gate_per == 1) inv *= 1.0f / (1.0f + expf(-gr[head]));
-            const bool each = gr != nullptr && gate_per > 1;
             bf16* dst = out + (size_t)t * out_stride + (size_t)head * vd;
-#pragma unroll 1
+#pragma unroll
             for (int c = 0; c < OC / 32; c++) {
                 const int col = hf * OC + c * 32;
                 float v[32];
@@ -341,12 +365,7 @@ attn_sink_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         if (col + e >= vd) break;
                         float w[8];
 #pragma unroll
-                        for (int k = 0; k < 8; k++) w[k] = v[e + k] * inv;
-                        if (each) {
-                            const float* ge = gr + (size_t)head * vd + col + e;
-#pragma unroll
-                            for (int k = 0; k < 8; k++) w[k] *= 1.0f / (1.0f + expf(-ge[k]));
-                        }
+                        for (int k = 0; k < 8; k++) w[k] = v[e + k] * inv * gv[c * 32 + e + k];
                         uint4 o4;
                         o4.x = pack_bf16_pair(w[0], w[1]);
                         o4.y = pack_bf16_pair(w[2], w[3]);
