@@ -74,6 +74,20 @@ int tc_make_map(CUtensorMap* map, const void* base, long long rows, long long co
     return 0;
 }
 
+int tc_make_map_blocks(CUtensorMap* map, const void* base, long long rows, long long blocks, int box_rows, int box_blocks) {
+    EncodeTiledFn enc = get_encode();
+    if (!enc) return hb_fail("gemm_tc: cuTensorMapEncodeTiled is not available from this driver");
+    cuuint64_t dims[3] = {TC_BK, (cuuint64_t)rows, (cuuint64_t)blocks};
+    cuuint64_t strides[2] = {TC_BK * 2, (cuuint64_t)rows * TC_BK * 2};
+    cuuint32_t box[3] = {TC_BK, (cuuint32_t)box_rows, (cuuint32_t)box_blocks};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, (void*)base, dims, strides, box, estr,
+                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                     CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return hb_fail("gemm_tc: tensor map encode failed with code %d (%lld rows, %lld column blocks)", (int)r, rows, blocks);
+    return 0;
+}
+
 int tc_make_out_map(CUtensorMap* map, const void* base, int elem_bytes, long long rows, long long cols, long long ld,
                     int box_rows, int box_cols) {
     EncodeTiledFn enc = get_encode();

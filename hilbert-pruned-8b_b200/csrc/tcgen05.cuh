@@ -50,6 +50,12 @@ __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map
         ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1)
         : "memory");
 }
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, uint32_t bar, int c0, int c1, int c2) {
+    asm volatile(
+        "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+        ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1), "r"(c2)
+        : "memory");
+}
 // fetches a tensor map (a kernel parameter) into the descriptor cache ahead of its first use
 __device__ __forceinline__ void tma_prefetch_map(const CUtensorMap* map) {
     asm volatile("prefetch.tensormap [%0];" ::"l"(map) : "memory");
@@ -490,6 +496,9 @@ __device__ __forceinline__ void tc_emit_flat(const TcParams& p, int m0, int n0, 
 // Tensor map of a row-major bf16 matrix [rows, cols] with row stride ld (elements): boxes of
 // box_rows x 64 elements, 128-byte swizzle, zeros outside.
 int tc_make_map(CUtensorMap* map, const void* base, long long rows, long long cols, long long ld, int box_rows);
+// Tensor map of a bf16 matrix stored in column blocks, [block][rows][64 columns]: boxes of box_blocks x box_rows x 64 elements, so
+// that one copy brings several column blocks of some rows, each as a tile of its own; zeros outside.
+int tc_make_map_blocks(CUtensorMap* map, const void* base, long long rows, long long blocks, int box_rows, int box_blocks);
 // Tensor map of a row-major output [rows, cols] of float32 (elem_bytes 4) or bfloat16 (2) with
 // row stride ld (elements), for stores of boxes of box_rows x box_cols elements, no swizzle.
 // The base must be 16-byte aligned and ld * elem_bytes a multiple of 16.

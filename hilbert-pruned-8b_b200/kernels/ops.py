@@ -1841,14 +1841,14 @@ class Ops:
         max_tiles = self.moe_max_tiles(entries, E, tile_rows)
         plan = workspace.buffer("moe.plan" + tag, (E + 1 + most + 1 + 2 * self.moe_max_tiles(most, E, 16),), torch.int32)
         offsets, order, tiles = plan[: E + 1], plan[E + 1: E + 1 + most], plan[E + 1 + most:]
-        act = workspace.buffer("moe.act" + tag, (most, F), h.dtype)
+        act = workspace.buffer("moe.act" + tag, (most, (F + 63) // 64 * 64 if umma else F), h.dtype)       # (umma: in column blocks of 64)
         down = workspace.buffer("moe.down" + tag, (most, W), torch.float32)
         s = self._stream()
         self._call("hb_moe_plan", experts.data_ptr(), entries, E, tile_rows, offsets.data_ptr(), order.data_ptr(), tiles.data_ptr(), s)
         unit_code = {"gelu": 2, "clamped_glu": 1, "silu_glu": 3}[unit]
         in_weights = weights.data_ptr() if weigh == "input" else None
         if umma:
-            rows = workspace.buffer("moe.rows" + tag, (most, W), h.dtype)
+            rows = workspace.buffer("moe.rows" + tag, (most, (W + 63) // 64 * 64), h.dtype)
             self._call("hb_moe_gather", h.data_ptr(), _rows(h, "expert input"), offsets.data_ptr(), E, order.data_ptr(), top, rows.data_ptr(), entries, W, s)
             self._call("hb_moe_tc", rows.data_ptr(), entries, w_gate.data.data_ptr(), E, offsets.data_ptr(),
                        order.data_ptr(), tiles.data_ptr(), max_tiles, tile_rows, unit_code, act.data_ptr(), F, F, W, float(limit), float(alpha), in_weights,
